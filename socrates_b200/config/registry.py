@@ -16,6 +16,7 @@ from .loletar import LoletarConfig
 from .magedra import MagedraConfig
 from .qwen3 import ConfigError, Qwen3Config
 from .samerax import SameraxConfig
+from .samovik import SamovikConfig
 
 _ARCHITECTURES: Dict[str, Any] = {}
 
@@ -63,3 +64,4 @@ register_architecture(BofusunConfig.architecture, BofusunConfig)
 register_architecture(LoletarConfig.architecture, LoletarConfig)
 register_architecture(SameraxConfig.architecture, SameraxConfig)
 register_architecture(MagedraConfig.architecture, MagedraConfig)
+register_architecture(SamovikConfig.architecture, SamovikConfig)

@@ -7,6 +7,7 @@
 //                   residual[r] = v ;  out[m] = v / sqrt(mean(v^2) + eps) * gain    (if out)
 //                   (out with a null gain: out[m] = v, the stream itself in the model dtype, for
 //                   blocks whose branches read the stream without a norm in front)
+//                   (with tanh_alpha: out[m] = tanh(alpha v) * gain + tanh_bias, nothing is averaged)
 //   normed_mean:    out[r] = scale * sum_t unit_rms(sum_s x_t[s][r]) * gain_t       (t < 2)
 //   bias_act:       out[r][f] = act(sum_s in[s][r][f] + bias[f])
 #include <math.h>
@@ -33,6 +34,8 @@ struct FoldArgs {
     int d;
     float eps;
     int write_residual;
+    const float* tanh_alpha;   // [1] or null: the out rows are tanh(alpha v) * gain + tanh_bias
+    const float* tanh_bias;    // [d]
 };
 
 template <typename T>
@@ -82,6 +85,12 @@ __global__ void __launch_bounds__(256) fold_rmsnorm_kernel(FoldArgs a) {
     T* o = (T*)a.out + (size_t)m * d;
     if (a.gain == nullptr) {
         for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = from_float<T>(row[i]);
+        return;
+    }
+    if (a.tanh_alpha != nullptr) {
+        const float alpha = *a.tanh_alpha;
+        for (int i = threadIdx.x; i < d; i += blockDim.x)
+            o[i] = from_float<T>(fmaf(tanhf(alpha * row[i]), a.gain[i], a.tanh_bias[i]));
         return;
     }
     const float total = block_sum(ss, scratch);
@@ -155,13 +164,20 @@ __global__ void __launch_bounds__(512) fold_rmsnorm_vec_kernel(FoldArgs a) {
         ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
     if (a.out == nullptr) return;
-    const bool normed = a.gain != nullptr;
+    const bool squash = a.tanh_alpha != nullptr, normed = a.gain != nullptr && !squash;
+    const float alpha = squash ? *a.tanh_alpha : 0.f;
     const float rinv = normed ? 1.0f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps) : 1.0f;
     T* o = (T*)a.out + (size_t)m * a.d;
     for (int i = threadIdx.x; i < d4; i += blockDim.x) {
         const float4 v = row4[i];
         const float4 g = normed ? __ldg(reinterpret_cast<const float4*>(a.gain) + i) : make_float4(1.f, 1.f, 1.f, 1.f);
-        const float x0 = v.x * rinv * g.x, x1 = v.y * rinv * g.y, x2 = v.z * rinv * g.z, x3 = v.w * rinv * g.w;
+        float x0 = v.x * rinv * g.x, x1 = v.y * rinv * g.y, x2 = v.z * rinv * g.z, x3 = v.w * rinv * g.w;
+        if (squash) {
+            const float4 c = __ldg(reinterpret_cast<const float4*>(a.gain) + i);
+            const float4 b = __ldg(reinterpret_cast<const float4*>(a.tanh_bias) + i);
+            x0 = fmaf(tanhf(alpha * v.x), c.x, b.x); x1 = fmaf(tanhf(alpha * v.y), c.y, b.y);
+            x2 = fmaf(tanhf(alpha * v.z), c.z, b.z); x3 = fmaf(tanhf(alpha * v.w), c.w, b.w);
+        }
         if constexpr (sizeof(T) == 2) {
             __nv_bfloat162 lo = __floats2bfloat162_rn(x0, x1), hi = __floats2bfloat162_rn(x2, x3);
             uint2 pk;
@@ -221,6 +237,7 @@ __device__ __forceinline__ float activation(float z, int act) {
         case 1: { const float p = fmaxf(z, 0.f); return p * p; }                       // relu squared
         case 2: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));   // gelu (tanh form)
         case 3: return z / (1.0f + expf(-z));                                          // silu
+        case 4: return tanhf(z);
         default: return z;
     }
 }
@@ -250,10 +267,12 @@ __global__ void __launch_bounds__(256) bias_act_kernel(T* __restrict__ out, cons
 extern "C" int sb_fold_rmsnorm(float* residual, const float* delta, int S, long long delta_stride,
                                const float* branch_bias, const float* branch_gain, float branch_eps,
                                const float* add_rows, const float* add_vec, const float* gain, void* out,
-                               const int* row_index, int M, int d, float eps, int out_dtype,
-                               cudaStream_t stream) {
+                               const int* row_index, int M, int d, float eps, const float* tanh_alpha,
+                               const float* tanh_bias, int out_dtype, cudaStream_t stream) {
     SB_REQUIRE(M >= 0 && d > 0 && S >= 0, "fold_rmsnorm: bad sizes M=%d d=%d S=%d", M, d, S);
     SB_REQUIRE(S == 0 || delta != nullptr, "fold_rmsnorm: S=%d partial sums but no buffer", S);
+    SB_REQUIRE((tanh_alpha != nullptr) == (tanh_bias != nullptr) && (tanh_alpha == nullptr || gain != nullptr),
+               "fold_rmsnorm: tanh rows need alpha, a gain and a bias");
     if (M == 0) return 0;
     const size_t smem = (size_t)d * sizeof(float);
     SB_REQUIRE(smem <= 200 * 1024, "fold_rmsnorm: width %d does not fit one block's shared memory", d);
@@ -261,12 +280,13 @@ extern "C" int sb_fold_rmsnorm(float* residual, const float* delta, int S, long 
     a.residual = residual; a.delta = delta; a.S = S; a.delta_stride = (size_t)delta_stride;
     a.branch_bias = branch_bias; a.branch_gain = branch_gain; a.branch_eps = branch_eps;
     a.add_rows = add_rows; a.add_vec = add_vec; a.gain = gain; a.out = out; a.row_index = row_index;
-    a.d = d; a.eps = eps;
+    a.d = d; a.eps = eps; a.tanh_alpha = tanh_alpha; a.tanh_bias = tanh_bias;
     a.write_residual = row_index == nullptr &&
                        (S > 0 || branch_bias != nullptr || add_rows != nullptr || add_vec != nullptr);
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     const bool vec = d % 4 == 0 && delta_stride % 4 == 0 && aligned(residual) && aligned(delta) && aligned(branch_bias) &&
-                     aligned(branch_gain) && aligned(add_rows) && aligned(add_vec) && aligned(gain) && aligned(out);
+                     aligned(branch_gain) && aligned(add_rows) && aligned(add_vec) && aligned(gain) && aligned(tanh_bias) &&
+                     aligned(out);
     if (vec) {
         int threads = ((d / 4 + 31) / 32) * 32;
         if (threads > 512) threads = 512;
@@ -318,7 +338,7 @@ extern "C" int sb_normed_mean(float* out, const float* x0, int S0, long long str
 // in: [N, F] in the model dtype, or (parts != null) float32 partial sums [S, N, F].
 extern "C" int sb_bias_act(void* out, const void* in, const float* parts, int S, long long part_stride,
                            const float* bias, int N, int F, int act, int dtype, cudaStream_t stream) {
-    SB_REQUIRE(N >= 0 && F > 0 && act >= 0 && act <= 3, "bias_act: bad sizes N=%d F=%d or activation %d", N, F, act);
+    SB_REQUIRE(N >= 0 && F > 0 && act >= 0 && act <= 4, "bias_act: bad sizes N=%d F=%d or activation %d", N, F, act);
     SB_REQUIRE((in != nullptr) != (parts != nullptr), "bias_act: one input, a matrix or partial sums");
     if (N == 0) return 0;
     const size_t total = (size_t)N * F;

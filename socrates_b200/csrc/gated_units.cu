@@ -7,6 +7,7 @@
 //                  (or y = x without a gain), written to one or two places
 //   head_matmul:   y[n, h, :] = W_h x[n, h, :]  or  W_h^T x[n, h, :],  W_h = rows h*A .. h*A + A - 1 of W [H*A, B]
 //   scale:         x *= c
+//   gelu_lookup:   out[n, i] = gelu(in[n, i]) * table[id_n, first + i]        (gelu in its tanh form)
 //   latent_write:  per token: c = rmsnorm(latent) * w; the shared key part and every query head's first `dr`
 //                  dims are turned by the token's position; the row [turned key part | c] goes into the key
 //                  page and c into the value page (one head), the queries are turned in place
@@ -79,6 +80,32 @@ __global__ void __launch_bounds__(256) scale_kernel(float* __restrict__ x, size_
     sb::pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
         x[i] *= c;
+}
+
+// A negative id -1 - j stands for feedback[j], a token that an earlier kernel on the stream wrote.
+template <typename T>
+__global__ void __launch_bounds__(256) gelu_lookup_kernel(T* __restrict__ out, const T* __restrict__ in,
+                                                          const float* __restrict__ parts, int S, size_t part_stride,
+                                                          const T* __restrict__ table, long long table_stride, int first,
+                                                          const int* __restrict__ ids, const int* __restrict__ feedback,
+                                                          int V, int F, size_t total) {
+    sb::pdl_launch_dependents();
+    sb::pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t n = i / F;
+        const int f = (int)(i - n * F);
+        int id = ids[n];
+        if (id < 0 && feedback != nullptr) id = feedback[-1 - id];
+        id = id < 0 ? 0 : (id >= V ? V - 1 : id);
+        float z = 0.f;
+        if (parts) {
+            for (int s = 0; s < S; ++s) z += parts[s * part_stride + i];
+        } else {
+            z = to_float(in[i]);
+        }
+        const float g = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+        out[i] = from_float<T>(g * to_float(table[(size_t)id * table_stride + first + f]));
+    }
 }
 
 constexpr int MAX_SEGMENTS = 4;
@@ -292,6 +319,26 @@ extern "C" int sb_scale(float* x, long long total, float c, cudaStream_t stream)
     SB_REQUIRE(total >= 0, "scale: a negative size");
     if (total == 0) return 0;
     sb::launch(scale_kernel, dim3(blocks_for((size_t)total)), dim3(256), 0, stream, x, (size_t)total, c);
+    SB_LAUNCH_CHECK();
+}
+
+extern "C" int sb_gelu_lookup(void* out, const void* in, const float* parts, int S, long long part_stride,
+                              const void* table, long long table_stride, int first, const int* ids, const int* feedback,
+                              int V, int N, int F, int dtype, cudaStream_t stream) {
+    SB_REQUIRE(N >= 0 && F > 0 && V > 0 && first >= 0 && first + F <= table_stride,
+               "gelu_lookup: columns %d..%d of table rows of %lld", first, first + F, table_stride);
+    SB_REQUIRE((in != nullptr) != (parts != nullptr), "gelu_lookup: one input, a matrix or partial sums");
+    if (N == 0) return 0;
+    const size_t total = (size_t)N * F;
+    if (dtype == SB_F32)
+        sb::launch(gelu_lookup_kernel<float>, dim3(blocks_for(total)), dim3(256), 0, stream, (float*)out, (const float*)in, parts,
+                   S, (size_t)part_stride, (const float*)table, table_stride, first, ids, feedback, V, F, total);
+    else if (dtype == SB_BF16)
+        sb::launch(gelu_lookup_kernel<__nv_bfloat16>, dim3(blocks_for(total)), dim3(256), 0, stream, (__nv_bfloat16*)out,
+                   (const __nv_bfloat16*)in, parts, S, (size_t)part_stride, (const __nv_bfloat16*)table, table_stride, first,
+                   ids, feedback, V, F, total);
+    else
+        SB_REQUIRE(false, "gelu_lookup: unknown dtype %d", dtype);
     SB_LAUNCH_CHECK();
 }
 

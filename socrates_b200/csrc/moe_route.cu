@@ -7,6 +7,9 @@
 //                largest c; only the `keep` best groups stay (the others' c count as -inf)
 //                the `top` largest c are chosen; their weights are s (no correction, not renormalized)
 //                weights[n][e] = s_e for chosen e, else 0 ;  ids[n][k], picked[n][k] = the choices, best first
+//   route, chosen: the `top` largest of z + bias are chosen; their weights are the softmax over these only
+//   glu_clamp:   all experts' gated units and the shared one's in one pass, scaled on the way out:
+//                g = min(pg, limit) ,  u = clamp(pu, -limit, limit) ,  act = g * sigmoid(alpha g) * (u + offset) * weight
 //   scale:       act[n][e*F + f] *= weights[n][e]                (all experts' activations side by side)
 //   passthrough: slab[n][:] = x[n][:] * sum of weights[n][e] over e >= first_identity
 //                (router outputs past the real experts stand for "the input itself")
@@ -107,6 +110,137 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(
             c[bi] = NAN;                         // taken
         }
         __syncwarp();
+    }
+}
+
+// Weights from the chosen logits only: a warp per token, ties to the lower index.
+__global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_chosen_kernel(
+    const float* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ weights, int* __restrict__ ids,
+    float* __restrict__ picked, int N, int E, int top) {
+    sb::pdl_launch_dependents();
+    extern __shared__ float rsm[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* c = rsm + (size_t)warp * 2 * E;                  // open logits
+    float* w = c + E;                                       // weights
+    const int n = blockIdx.x * ROUTE_WARPS + warp;
+    sb::pdl_wait();
+    if (n >= N) return;
+    for (int e = lane; e < E; e += 32) {
+        c[e] = logits[(size_t)n * E + e] + (bias ? bias[e] : 0.f);
+        w[e] = 0.f;
+    }
+    __syncwarp();
+    float best = 0.f, sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float bv = -INFINITY;
+        int bi = 0x7fffffff;
+        for (int e = lane; e < E; e += 32) {
+            const float v = c[e];
+            if (!isnan(v) && (v > bv || (bi == 0x7fffffff && w[e] == 0.f))) { bv = v; bi = e; }
+        }
+        warp_argmax(bv, bi);
+        if (k == 0) best = bv;
+        const float p = expf(bv - best);
+        sum += p;
+        if (lane == 0 && bi < E) {
+            ids[(size_t)n * top + k] = bi;
+            picked[(size_t)n * top + k] = p;
+            w[bi] = p;
+            c[bi] = NAN;                                     // taken
+        }
+        __syncwarp();
+    }
+    const float inv = 1.0f / sum;
+    for (int e = lane; e < E; e += 32) weights[(size_t)n * E + e] = w[e] * inv;
+    for (int k = lane; k < top; k += 32) picked[(size_t)n * top + k] *= inv;
+}
+
+// Column f < experts * F belongs to expert f / F; the columns from there on to the shared expert, whose weight is
+// one.  An expert that was not chosen is not read: its activations are zero.
+struct MoeGluArgs {
+    const void* in;            // [N, 2W] in T (gates, then values), or null
+    const float* parts;        // [S, N, 2W]
+    int S;
+    size_t part_stride;
+    const float* weights;      // [N, E_total]
+    void* out;                 // [N, W] in T
+    int W, E_total, experts, F;
+    float limit, shared_limit, alpha, offset;
+};
+
+__device__ __forceinline__ float glu_clamped(float g, float u, float limit, float alpha, float offset) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + offset);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) moe_glu_clamp_kernel(MoeGluArgs a, size_t total) {
+    sb::pdl_launch_dependents();
+    sb::pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t n = i / a.W;
+        const int f = (int)(i - n * a.W), e = f / a.F;
+        const bool shared = e >= a.experts;
+        const float w = shared ? 1.f : a.weights[n * a.E_total + e];
+        float y = 0.f;
+        if (w != 0.f) {
+            const size_t at = n * 2 * a.W + f;
+            float g = 0.f, u = 0.f;
+            if (a.parts) {
+                for (int s = 0; s < a.S; ++s) { g += a.parts[s * a.part_stride + at]; u += a.parts[s * a.part_stride + at + a.W]; }
+            } else {
+                g = to_float(((const T*)a.in)[at]);
+                u = to_float(((const T*)a.in)[at + a.W]);
+            }
+            y = glu_clamped(g, u, shared ? a.shared_limit : a.limit, a.alpha, a.offset) * w;
+        }
+        ((T*)a.out)[i] = from_float<T>(y);
+    }
+}
+
+// F and W multiples of the 16-byte vector: a thread takes one vector, whose elements share their expert.
+template <typename T>
+__global__ void __launch_bounds__(256) moe_glu_clamp_vec_kernel(MoeGluArgs a, size_t packs) {
+    sb::pdl_launch_dependents();
+    sb::pdl_wait();
+    constexpr int VEC = Vec16<T>::N;
+    const int per_row = a.W / VEC;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < packs; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t n = i / per_row;
+        const int f = (int)(i - n * per_row) * VEC, e = f / a.F;
+        const bool shared = e >= a.experts;
+        const float w = shared ? 1.f : a.weights[n * a.E_total + e];
+        T* out = (T*)a.out + n * a.W + f;
+        if (w == 0.f) {
+            *reinterpret_cast<uint4*>(out) = make_uint4(0u, 0u, 0u, 0u);
+            continue;
+        }
+        const float limit = shared ? a.shared_limit : a.limit;
+        float g[VEC], u[VEC];
+        if (a.parts) {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) g[j] = u[j] = 0.f;
+            for (int s = 0; s < a.S; ++s) {
+                const float* p = a.parts + s * a.part_stride + n * 2 * a.W + f;
+#pragma unroll
+                for (int j = 0; j < VEC; j += 4) {
+                    const float4 x = *reinterpret_cast<const float4*>(p + j), y = *reinterpret_cast<const float4*>(p + a.W + j);
+                    g[j] += x.x; g[j + 1] += x.y; g[j + 2] += x.z; g[j + 3] += x.w;
+                    u[j] += y.x; u[j + 1] += y.y; u[j + 2] += y.z; u[j + 3] += y.w;
+                }
+            }
+        } else {
+            Vec16<T> gv, uv;
+            gv.load((const T*)a.in + n * 2 * a.W + f);
+            uv.load((const T*)a.in + n * 2 * a.W + a.W + f);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) { g[j] = gv.get(j); u[j] = uv.get(j); }
+        }
+        alignas(16) T y[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) y[j] = from_float<T>(glu_clamped(g[j], u[j], limit, a.alpha, a.offset) * w);
+        *reinterpret_cast<uint4*>(out) = *reinterpret_cast<const uint4*>(y);
     }
 }
 
@@ -248,6 +382,48 @@ extern "C" int sb_moe_route(const float* logits, const float* correction, float*
     if (N == 0) return 0;
     sb::launch(moe_route_kernel, dim3((N + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream,
                logits, correction, weights, ids, picked, N, E, groups, keep, top);
+    SB_LAUNCH_CHECK();
+}
+
+extern "C" int sb_moe_route_chosen(const float* logits, const float* bias, float* weights, int* ids, float* picked, int N,
+                                   int E, int top, cudaStream_t stream) {
+    SB_REQUIRE(N >= 0 && E > 0 && top >= 1 && top <= E, "moe_route_chosen: bad sizes N=%d E=%d top=%d", N, E, top);
+    const size_t smem = (size_t)ROUTE_WARPS * 2 * E * sizeof(float);
+    SB_REQUIRE(smem <= 48 * 1024, "moe_route_chosen: %d router outputs do not fit a block's shared memory", E);
+    if (N == 0) return 0;
+    sb::launch(moe_route_chosen_kernel, dim3((N + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream,
+               logits, bias, weights, ids, picked, N, E, top);
+    SB_LAUNCH_CHECK();
+}
+
+// in [N, 2W] in the model dtype (or parts float32 [S, N, 2W]), W = experts * F + shared columns.
+extern "C" int sb_moe_glu_clamp(void* out, const void* in, const float* parts, int S, long long part_stride,
+                                const float* weights, int N, int W, int E_total, int experts, int F, float limit,
+                                float shared_limit, float alpha, float offset, int dtype, cudaStream_t stream) {
+    SB_REQUIRE(N >= 0 && experts > 0 && experts <= E_total && F > 0 && W >= experts * F,
+               "moe_glu_clamp: bad sizes N=%d experts=%d/%d F=%d W=%d", N, experts, E_total, F, W);
+    SB_REQUIRE(limit > 0.f && shared_limit > 0.f, "moe_glu_clamp: clamps at %f and %f", limit, shared_limit);
+    SB_REQUIRE((in != nullptr) != (parts != nullptr), "moe_glu_clamp: one input, a matrix or partial sums");
+    if (N == 0) return 0;
+    MoeGluArgs a;
+    a.in = in; a.parts = parts; a.S = S; a.part_stride = (size_t)part_stride; a.weights = weights; a.out = out; a.W = W;
+    a.E_total = E_total; a.experts = experts; a.F = F; a.limit = limit; a.shared_limit = shared_limit; a.alpha = alpha;
+    a.offset = offset;
+    const size_t total = (size_t)N * W;
+    const int vec = dtype == SB_BF16 ? 8 : 4;
+    const bool wide = F % vec == 0 && W % vec == 0 && part_stride % 4 == 0 &&
+                      ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(parts) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const size_t items = wide ? total / vec : total;
+    const int blocks = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
+    if (dtype == SB_F32) {
+        if (wide) sb::launch(moe_glu_clamp_vec_kernel<float>, dim3(blocks), dim3(256), 0, stream, a, items);
+        else sb::launch(moe_glu_clamp_kernel<float>, dim3(blocks), dim3(256), 0, stream, a, items);
+    } else if (dtype == SB_BF16) {
+        if (wide) sb::launch(moe_glu_clamp_vec_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, a, items);
+        else sb::launch(moe_glu_clamp_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, a, items);
+    } else {
+        SB_REQUIRE(false, "moe_glu_clamp: unknown dtype %d", dtype);
+    }
     SB_LAUNCH_CHECK();
 }
 

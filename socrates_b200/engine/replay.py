@@ -30,7 +30,7 @@ import sys
 from pathlib import Path
 from typing import Dict, List
 
-MAX_LIVE = 8
+MAX_LIVE = 4
 
 
 def main(argv=None) -> int:

@@ -48,7 +48,7 @@ _SIGNATURES = {
     "sb_attention_decode_stream": [P, P, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "sb_attention_tcgen05_supports": [I, I, I, I],
     "sb_attention_prefill_tcgen05": [P, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, P, P, LL, I, I, F, I, P, P],
-    "sb_fold_rmsnorm": [P, P, I, LL, P, P, F, P, P, P, P, P, I, I, F, I, P],
+    "sb_fold_rmsnorm": [P, P, I, LL, P, P, F, P, P, P, P, P, I, I, F, P, P, I, P],
     "sb_normed_mean": [P, P, I, LL, P, P, I, LL, P, I, I, F, F, P],
     "sb_bias_act": [P, P, P, I, LL, P, I, I, I, I, P],
     "sb_short_conv": [P, LL, P, P, P, I, P, I, I, I, P, P, P, I, I, I, P, P, P, P, P, P, P, I, P],
@@ -77,6 +77,13 @@ _SIGNATURES = {
     "sb_gated_linear_attention": [P, P, LL, I, I, I, P, P, P, P, P, P, I, I, I, I, F, I, P, I, I, P, P],
     "sb_glu_clamp": [P, P, P, I, LL, P, P, I, I, F, F, F, I, P],
     "sb_scale": [P, LL, F, P],
+    "sb_gelu_lookup": [P, P, P, I, LL, P, LL, I, P, P, I, I, I, I, P],
+    "sb_linear_recurrence_supports": [I, I],
+    "sb_linear_recurrence": [P] + [P, I, LL, LL, I] * 4 + [P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, P, P, I, P],
+    "sb_norm_gate": [P, P, P, I, LL, LL, I, P, I, I, I, F, I, I, P],
+    "sb_token_shift_mix": [P, P, P, P, P, I, I, I, I, P],
+    "sb_moe_route_chosen": [P, P, P, P, P, I, I, I, P],
+    "sb_moe_glu_clamp": [P, P, P, I, LL, P, I, I, I, I, I, F, F, F, F, I, P],
     "sb_segment_norm": [P, LL, I, P, P, P, P, P, P, P, P, P, F, I, I, P],
     "sb_head_matmul": [P, LL, I, I, P, LL, I, I, P, I, I, I, I, I, I, I, P],
     "sb_latent_write": [P, LL, I, I, I, I, P, F, P, I, P, I, F, P, P, P, I, I, P, P, I, I, P],

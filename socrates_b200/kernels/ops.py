@@ -506,17 +506,19 @@ def attention_prefill_tcgen05(out: torch.Tensor, q: torch.Tensor, k_pool: torch.
 # ---------------------------------------------------------------------------------------------
 # Kernels of blocks that norm a branch before it joins the residual, and of recurrent mixers.
 
-ACTIVATIONS = {"identity": 0, "relu_squared": 1, "gelu_tanh": 2, "silu": 3}
+ACTIVATIONS = {"identity": 0, "relu_squared": 1, "gelu_tanh": 2, "silu": 3, "tanh": 4}
 
 
 def fold_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: Optional[torch.Tensor],
                  out: Optional[torch.Tensor], eps: float, row_index: Optional[torch.Tensor] = None,
                  branch_bias: Optional[torch.Tensor] = None, branch_gain: Optional[torch.Tensor] = None,
                  branch_eps: float = 0.0, add_rows: Optional[torch.Tensor] = None,
-                 add_vec: Optional[torch.Tensor] = None) -> None:
+                 add_vec: Optional[torch.Tensor] = None, tanh_alpha: Optional[torch.Tensor] = None,
+                 tanh_bias: Optional[torch.Tensor] = None) -> None:
     """b = sum(delta, 0) + branch_bias; with `branch_gain` b = b / sqrt(mean(b^2) + branch_eps) * branch_gain;
     residual += b + add_rows + add_vec; out = residual / sqrt(mean(residual^2) + eps) * gain
-    (gain None with an out: out = residual, rounded to out's dtype).
+    (gain None with an out: out = residual, rounded to out's dtype; with `tanh_alpha`, float32 of one element,
+    and `tanh_bias` [d]: out = tanh(alpha * residual) * gain + bias).
 
     residual float32 [N, d]; delta float32 [S, N, d] or None; the gains, the bias and add_vec float32 [d];
     add_rows float32 [N, d]; out [M, d] in float32 or bfloat16, or None (only the residual moves on).  With
@@ -530,9 +532,14 @@ def fold_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: Op
         if delta.dim() != 3 or delta.shape[1:] != (N, d):
             raise KernelError(f"delta must be [S, {N}, {d}], got {tuple(delta.shape)}")
         S, stride = delta.shape[0], N * d
-    for t, nm in ((gain, "gain"), (branch_bias, "branch_bias"), (branch_gain, "branch_gain"), (add_vec, "add_vec")):
+    for t, nm in ((gain, "gain"), (branch_bias, "branch_bias"), (branch_gain, "branch_gain"), (add_vec, "add_vec"),
+                  (tanh_bias, "tanh_bias")):
         if t is not None:
             _want(t, nm, torch.float32, (d,))
+    if tanh_alpha is not None:
+        _want(tanh_alpha, "tanh_alpha", torch.float32)
+        if tanh_alpha.numel() != 1:
+            raise KernelError(f"tanh_alpha must be one value, got {tuple(tanh_alpha.shape)}")
     if add_rows is not None:
         _want(add_rows, "add_rows", torch.float32, (N, d))
     M = N
@@ -546,7 +553,8 @@ def fold_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: Op
     lib = library()
     check(lib, lib.sb_fold_rmsnorm(_ptr(residual), _ptr(delta), S, stride, _ptr(branch_bias), _ptr(branch_gain),
                                    float(branch_eps), _ptr(add_rows), _ptr(add_vec), _ptr(gain), _ptr(out),
-                                   _ptr(row_index), M, d, float(eps), code, _stream()), "fold_rmsnorm")
+                                   _ptr(row_index), M, d, float(eps), _ptr(tanh_alpha), _ptr(tanh_bias), code, _stream()),
+          "fold_rmsnorm")
 
 
 def normed_mean(out: torch.Tensor, x0: torch.Tensor, gain0: torch.Tensor, x1: torch.Tensor, gain1: torch.Tensor,
@@ -1396,3 +1404,187 @@ def attention_talk_dense_step(step: int, q, k_pool, v_pool, table_row, Kc, Vt, Q
                                            gate_stride, _ptr(talk), num_heads, Hkv, Dk, Dv, BS, int(C), int(Cp), int(n0),
                                            int(nb), int(pos0), int(window), float(scale), _stream()),
           "attention_talk_dense")
+
+
+# ---------------------------------------------------------------------------------------------
+# Recurrences with a matrix state per head; routing by the chosen logits; a per-layer token input.
+
+def _rows(t: torch.Tensor, N: int, columns: int, first: int, dtype: torch.dtype, name: str):
+    """(pointer, S, part stride, row stride, first column) of a matrix [N, >= first + columns] in `dtype`, or of
+    float32 partial sums [S, N, >= first + columns]."""
+    if not t.is_cuda or t.stride(-1) != 1:
+        raise KernelError(f"{name} must be a CUDA tensor with unit column stride")
+    if t.dim() == 3:
+        if t.dtype != torch.float32 or t.shape[1] != N or first < 0 or t.shape[2] < first + columns:
+            raise KernelError(f"{name} must be float32 [S, {N}, >= {first + columns}], got {t.dtype} {tuple(t.shape)}")
+        return t.data_ptr(), t.shape[0], t.stride(0), t.stride(1), int(first)
+    if t.dim() != 2 or t.dtype != dtype or t.shape[0] != N or first < 0 or t.shape[1] < first + columns:
+        raise KernelError(f"{name} must be {dtype} [{N}, >= {first + columns}], got {t.dtype} {tuple(t.shape)}")
+    return t.data_ptr(), 0, 0, t.stride(0), int(first)
+
+
+def linear_recurrence_supports(key_dim: int, value_dim: int) -> bool:
+    return bool(library().sb_linear_recurrence_supports(int(key_dim), int(value_dim)))
+
+
+def linear_recurrence_segment(N: int, R: int) -> int:
+    """Tokens per segment for a step of N tokens from R requests: a function of the step's shape alone.  A step
+    whose longest portion fits one segment is one launch; otherwise the portions run as at most 16 + R segments
+    of at least 64 tokens."""
+    return max(64, -(-N // 16))
+
+
+def linear_recurrence_scratch(N: int, R: int, H: int, D: int, Dv: int) -> Tuple[int, int]:
+    """float32 elements of (segment states, segment decay products) the segments of a step need (0: none)."""
+    seg = linear_recurrence_segment(N, R)
+    if N - R + 1 <= seg:
+        return 0, 0
+    slots = 2 * (N // seg)                   # segments of requests that have more than one
+    return slots * H * D * Dv, slots * H * D
+
+
+def linear_recurrence(out: torch.Tensor, q, k, v, state: torch.Tensor, seq_starts: torch.Tensor, seq_rows: torch.Tensor,
+                      dtype: torch.dtype, decay: Optional[torch.Tensor] = None, raw_decay=None,
+                      decay_base: Optional[torch.Tensor] = None, bonus: Optional[torch.Tensor] = None,
+                      silu_qk: bool = False, silu_v: bool = False, seg_len: Optional[int] = None,
+                      seg_state: Optional[torch.Tensor] = None, seg_prod: Optional[torch.Tensor] = None) -> None:
+    """Every request's tokens of the step, in order, through its state slot: S <- diag(w) S + k v^T per head, with
+    o = S^T q after the write, or (`bonus` float32 [H*D]) o = (S + diag(bonus) k v^T)^T q before it.
+
+    q, k, v: (tensor, first column) with the heads side by side, a matrix in `dtype` or float32 partial sums;
+    `silu_qk`, `silu_v`: SiLU on the way in.  The decay w is the constant decay[h] (float32 [H]) or
+    exp(-exp(raw + decay_base)) per key channel with raw_decay = (float32 matrix or partial sums, first column).
+    state float32 [rows, H, D, Dv]; out float32 [N, H*Dv].  `seg_len` (default: `linear_recurrence_segment`): longer
+    portions run as segments side by side, which needs the scratch `linear_recurrence_scratch` gives."""
+    if state.dim() != 4:
+        raise KernelError(f"state must be [rows, H, D, Dv], got {tuple(state.shape)}")
+    _, H, D, Dv = state.shape
+    _want(state, "state", torch.float32)
+    N = out.shape[0]
+    _want(out, "out", torch.float32, (N, H * Dv))
+    R = seq_rows.numel()
+    _want(seq_starts, "seq_starts", torch.int32, (R + 1,))
+    _want(seq_rows, "seq_rows", torch.int32, (R,))
+    sources = [*_rows(q[0], N, H * D, q[1], dtype, "q"), *_rows(k[0], N, H * D, k[1], dtype, "k"),
+               *_rows(v[0], N, H * Dv, v[1], dtype, "v")]
+    if (decay is None) == (raw_decay is None):
+        raise KernelError("the decays are constants or come per token")
+    sources += [*_rows(raw_decay[0], N, H * D, raw_decay[1], torch.float32, "raw_decay")] if raw_decay is not None \
+        else [None, 0, 0, 0, 0]
+    if decay is not None:
+        _want(decay, "decay", torch.float32, (H,))
+    for t, nm in ((decay_base, "decay_base"), (bonus, "bonus")):
+        if t is not None:
+            _want(t, nm, torch.float32)
+            if t.numel() != H * D:
+                raise KernelError(f"{nm} must hold {H * D} values, got {tuple(t.shape)}")
+    longest = N - R + 1
+    seg_len = linear_recurrence_segment(N, R) if seg_len is None else int(seg_len)
+    several = longest > seg_len
+    if several:
+        slots = 2 * (N // seg_len)
+        for t, nm, n in ((seg_state, "seg_state", slots * H * D * Dv), (seg_prod, "seg_prod", slots * H * D)):
+            if t is None:
+                raise KernelError(f"segments of {seg_len} tokens need {nm}")
+            _want(t, nm, torch.float32)
+            if t.numel() < n:
+                raise KernelError(f"{nm} holds {t.numel()} of {n} values")
+    lib = library()
+    check(lib, lib.sb_linear_recurrence(_ptr(out), *sources, _ptr(decay), _ptr(decay_base), _ptr(bonus), int(silu_qk),
+                                        int(silu_v), _ptr(state), _ptr(seq_starts), _ptr(seq_rows), R, H, D, Dv, N,
+                                        seg_len, longest, _ptr(seg_state), _ptr(seg_prod), _code(dtype), _stream()),
+          "linear_recurrence", kernels=3 if several else 1)
+
+
+def norm_gate(out: torch.Tensor, x: torch.Tensor, gain: torch.Tensor, gate, groups: int, eps: float, act: str) -> None:
+    """out = x / sqrt(mean(x^2) + eps) * gain * act(gate), the mean over each of `groups` equal groups of columns;
+    x float32 [N, C], gain float32 [C], gate = (matrix in out's dtype or float32 partial sums, first column),
+    act "sigmoid" or "silu"."""
+    N, C = x.shape
+    _want(x, "x", torch.float32)
+    _want(out, "out", None, (N, C))
+    _want(gain, "gain", torch.float32, (C,))
+    if C % groups:
+        raise KernelError(f"{C} columns do not form {groups} equal groups")
+    lib = library()
+    check(lib, lib.sb_norm_gate(_ptr(out), _ptr(x), *_rows(gate[0], N, C, gate[1], out.dtype, "gate"), _ptr(gain), N, C,
+                                int(groups), float(eps), {"sigmoid": 0, "silu": 1}[act], _code(out.dtype), _stream()),
+          "norm_gate")
+
+
+def token_shift_mix(out: torch.Tensor, x: torch.Tensor, mu: torch.Tensor, last: torch.Tensor,
+                    token_rows: torch.Tensor) -> None:
+    """out[s] = x + (x' - x) * mu[s], x' the token before in the same request (`last` [rows, ..., d] for the first
+    token of a portion, not changed here); out [mixes, N, d] and x [N, d] share a dtype, mu float32 [mixes, d]."""
+    N, d = x.shape
+    _want(x, "x")
+    _want(mu, "mu", torch.float32)
+    mixes = mu.shape[0]
+    _want(mu, "mu", torch.float32, (mixes, d))
+    _want(out, "out", x.dtype, (mixes, N, d))
+    _want(last, "last", torch.float32)
+    if last.numel() != last.shape[0] * d:
+        raise KernelError(f"last must hold {d} values a row, got {tuple(last.shape)}")
+    _want(token_rows, "token_rows", torch.int32, (N,))
+    lib = library()
+    check(lib, lib.sb_token_shift_mix(_ptr(out), _ptr(x), _ptr(mu), _ptr(last), _ptr(token_rows), mixes, N, d,
+                                      _code(x.dtype), _stream()), "token_shift_mix")
+
+
+def moe_route_chosen(logits: torch.Tensor, bias: Optional[torch.Tensor], weights: torch.Tensor, ids: torch.Tensor,
+                     picked: torch.Tensor, top: int) -> None:
+    """Choose the `top` largest of logits + bias per token; weights float32 [N, E] gets the softmax over the chosen
+    ones at their places and 0 elsewhere, ids int32 / picked float32 [N, top] the choices best first."""
+    N, E = logits.shape
+    _want(logits, "logits", torch.float32)
+    if bias is not None:
+        _want(bias, "bias", torch.float32, (E,))
+    _want(weights, "weights", torch.float32, (N, E))
+    _want(ids, "ids", torch.int32, (N, top))
+    _want(picked, "picked", torch.float32, (N, top))
+    lib = library()
+    check(lib, lib.sb_moe_route_chosen(_ptr(logits), _ptr(bias), _ptr(weights), _ptr(ids), _ptr(picked), N, E, int(top),
+                                       _stream()), "moe_route_chosen")
+
+
+def moe_glu_clamp(out: torch.Tensor, x: torch.Tensor, weights: torch.Tensor, experts: int, inter: int, limit: float,
+                  shared_limit: float, alpha: float, offset: float) -> None:
+    """All experts' clamped gated units side by side, each times its token's weight (0: not computed), with a shared
+    expert's columns (weight one, a clamp of its own) behind them: out [N, W], W = experts * inter + shared columns;
+    x [N, 2W] (gates, then values) in out's dtype or float32 partial sums [S, N, 2W]; weights float32 [N, >= experts]."""
+    N, W = out.shape
+    _want(out, "out")
+    parts = x.dim() == 3
+    if parts:
+        _want(x, "x partial sums", torch.float32, (x.shape[0], N, 2 * W))
+    else:
+        _want(x, "x", out.dtype, (N, 2 * W))
+    _want(weights, "weights", torch.float32)
+    if weights.shape[0] != N or weights.shape[1] < experts or W < experts * inter:
+        raise KernelError(f"weights {tuple(weights.shape)} do not fit {experts} experts of {inter} in {W} columns")
+    lib = library()
+    check(lib, lib.sb_moe_glu_clamp(_ptr(out), None if parts else _ptr(x), _ptr(x) if parts else None,
+                                    x.shape[0] if parts else 0, N * 2 * W, _ptr(weights), N, W, weights.shape[1],
+                                    int(experts), int(inter), float(limit), float(shared_limit), float(alpha),
+                                    float(offset), _code(out.dtype), _stream()), "moe_glu_clamp")
+
+
+def gelu_lookup(out: torch.Tensor, x: torch.Tensor, table: torch.Tensor, first: int, ids: torch.Tensor,
+                feedback: Optional[torch.Tensor] = None) -> None:
+    """out[n, i] = gelu(x[n, i]) * table[ids[n], first + i] (gelu in its tanh form); x [N, F] in out's dtype or
+    float32 partial sums [S, N, F]; table [V, >= first + F] in out's dtype; ids as in `embed`."""
+    N, F_ = out.shape
+    _want(out, "out")
+    parts = x.dim() == 3
+    if parts:
+        _want(x, "x partial sums", torch.float32, (x.shape[0], N, F_))
+    else:
+        _want(x, "x", out.dtype, (N, F_))
+    _want(table, "table", out.dtype)
+    _want(ids, "ids", torch.int32, (N,))
+    if first < 0 or first + F_ > table.shape[1]:
+        raise KernelError(f"columns {first}..{first + F_} of a table of {table.shape[1]}")
+    lib = library()
+    check(lib, lib.sb_gelu_lookup(_ptr(out), None if parts else _ptr(x), _ptr(x) if parts else None,
+                                  x.shape[0] if parts else 0, N * F_, _ptr(table), table.stride(0), int(first), _ptr(ids),
+                                  _ptr(feedback), table.shape[0], N, F_, _code(out.dtype), _stream()), "gelu_lookup")

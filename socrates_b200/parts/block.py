@@ -87,6 +87,75 @@ class PreNormMixerBlock(PreNormBlock):
 register_part("arrangement", "pre_norm_mixer", lambda layer_spec, name="": PreNormMixerBlock(layer_spec))
 
 
+def stream_rows(ctx, stream: ResidualStream) -> torch.Tensor:
+    """The residual, with everything that waits on it added, as rows in the model dtype for a product that reads
+    the stream without a norm in front (the float32 engine reads the residual in place)."""
+    waiting = stream.pending is not None or stream.add_rows is not None or stream.add_vec is not None
+    if ctx.dtype == torch.float32:
+        if waiting:
+            fold_and_norm(stream, None, None, 0.0)
+        return stream.residual
+    out = ctx.buffers.take("stream_rows", stream.residual.shape[0], (stream.residual.shape[1],), ctx.dtype)
+    fold_and_norm(stream, None, out, 0.0)
+    return out
+
+
+class PreNormAfterBlock:
+    """A pre-norm layer that ends with a stream op: x = x + mixer(norm_0(x)); x = x + feed_forward(norm_1(x));
+    then the op named by the layer's params under "after" (None: nothing) acts on the stream.  A layer without a
+    feed-forward has one norm."""
+
+    def __init__(self, layer_spec):
+        want = 2 if layer_spec.feed_forward is not None else 1
+        if len(layer_spec.norms) != want:
+            raise ValueError(f"a pre_norm_after block with{'' if want == 2 else 'out'} a feed-forward has {want} norm(s)")
+        pre = layer_spec.prefix
+        self.norms = [build_part("norm", s, pre + s.name) for s in layer_spec.norms]
+        self.mixer = build_part("mixer", layer_spec.mixer, pre + layer_spec.mixer.name)
+        self.feed_forward = None
+        if layer_spec.feed_forward is not None:
+            self.feed_forward = build_part("feed_forward", layer_spec.feed_forward, pre + layer_spec.feed_forward.name)
+        after = layer_spec.params.get("after")
+        self.after = build_part("stream_op", after, pre + after.name) if after is not None else None
+
+    def parts(self):
+        return [*self.norms, self.mixer, *(p for p in (self.feed_forward, self.after) if p is not None)]
+
+    def parameters(self) -> Dict[str, ParamSpec]:
+        out: Dict[str, ParamSpec] = {}
+        for p in self.parts():
+            out.update(p.parameters())
+        return out
+
+    def bind(self, tensors: Mapping, dtype) -> None:
+        for p in self.parts():
+            p.bind(tensors, dtype)
+
+    @property
+    def supports_graph(self) -> bool:
+        return all(getattr(p, "supports_graph", True) for p in self.parts())
+
+    def cache_needs(self):
+        fn = getattr(self.mixer, "cache_needs", None)
+        return fn() if fn is not None else None
+
+    def streamed_weights(self):
+        return [w for p in (self.mixer, self.feed_forward, self.after) if p is not None
+                for w in getattr(p, "streamed_weights", list)()]
+
+    def forward(self, ctx, stream: ResidualStream, cache) -> None:
+        h = self.norms[0].apply(ctx, stream)
+        stream.pending = self.mixer.forward(ctx, h, cache)
+        if self.feed_forward is not None:
+            h = self.norms[1].apply(ctx, stream)
+            stream.pending = self.feed_forward.forward(ctx, h)
+        if self.after is not None:
+            self.after.apply(ctx, stream)
+
+
+register_part("arrangement", "pre_norm_after", lambda layer_spec, name="": PreNormAfterBlock(layer_spec))
+
+
 class SandwichBlock:
     """A block that norms every branch on both sides:
     x = x + norm_1b(mixer(norm_1(x))); x = x + norm_2b(feed_forward(norm_2(x))).
@@ -172,22 +241,11 @@ class BranchNormBlock(SandwichBlock):
             self.feed_forward = build_part("feed_forward", layer_spec.feed_forward,
                                            pre + layer_spec.feed_forward.name)
 
-    @staticmethod
-    def _stream_rows(ctx, stream: ResidualStream) -> torch.Tensor:
-        waiting = stream.pending is not None or stream.add_rows is not None or stream.add_vec is not None
-        if ctx.dtype == torch.float32:
-            if waiting:
-                fold_and_norm(stream, None, None, 0.0)
-            return stream.residual
-        out = ctx.buffers.take("stream_rows", stream.residual.shape[0], (stream.residual.shape[1],), ctx.dtype)
-        fold_and_norm(stream, None, out, 0.0)
-        return out
-
     def forward(self, ctx, stream: ResidualStream, cache) -> None:
-        h = self._stream_rows(ctx, stream)
+        h = stream_rows(ctx, stream)
         stream.pending = self._normed_on_entry(self.mixer.forward(ctx, h, cache), self.norms[0])
         if self.feed_forward is not None:
-            h = self._stream_rows(ctx, stream)
+            h = stream_rows(ctx, stream)
             stream.pending = self._normed_on_entry(self.feed_forward.forward(ctx, h), self.norms[1])
 
 

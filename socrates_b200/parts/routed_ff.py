@@ -12,6 +12,14 @@ and the choice are float32 in both engines.
 With `router: "table"` there is no router product at all: an integer table [vocab, top] names the experts of
 every token ID (no expert twice in a row), and each of them counts 1 / top.
 
+With `weighting: "chosen"` the experts are chosen by the logits themselves (plus `router.b` with `router_bias`)
+and weighed by the softmax over the chosen logits only.
+
+With `clamp` (`limit`, `alpha`, `offset`) an expert is the clamped gated unit instead:
+    g = min(W_gate x, limit) ,  u = clamp(W_up x, -limit, limit) ,  W_down (g * sigmoid(alpha g) * (u + offset))
+and `shared` (`intermediate_size`, `limit`) names one more such expert that runs for every token with weight one:
+its rows stand behind the experts' in both products.
+
 How it runs: all experts' gate/up matrices are one matrix [E * 2F, d] (rows interleaved as in the dense
 gated feed-forward, so the product's epilogue applies silu(gate) * up) and all down matrices one matrix
 [d, E * F].  The routing kernel leaves a dense float32 weight per (token, expert), zero where the expert
@@ -21,7 +29,10 @@ the branch's partial sums.  Nothing is read back and no shape depends on the cho
 recorded into graphs like any other; the price is that every expert is computed for every token, which
 costs nothing while a step streams the weights anyway (decoding) and E / top times the needed products
 for long prompt portions.
-Tensors: `<name>router`, `correction` (or `table`), `e<i>.gate`, `e<i>.up`, `e<i>.down`.
+For clamped experts gates and values are two halves of the first product and one kernel clamps, gates and
+scales all experts' units.
+Tensors: `<name>router`, `router.b`, `correction` (or `table`), `e<i>.gate`, `e<i>.up`, `e<i>.down`, `shared.gate`,
+`shared.up`, `shared.down`.
 """
 
 from __future__ import annotations
@@ -67,7 +78,24 @@ class RoutedFeedForward(Part):
             raise ValueError(f"{self.E} router outputs in {self.groups} groups of which {self.keep} stay")
         if not 1 <= self.top <= self.keep * (self.E // self.groups):
             raise ValueError(f"{self.top} choices among {self.keep * (self.E // self.groups)} open experts")
-        self.router = self.correction = self.table = None
+        self.weighting = str(p.get("weighting", "all"))       # softmax over "all" outputs or the "chosen" ones
+        if self.weighting not in ("all", "chosen"):
+            raise ValueError(f"weighting {self.weighting!r} is neither 'all' nor 'chosen'")
+        if self.weighting == "chosen" and (self.routing == "table" or self.groups > 1 or self.correction_tensor):
+            raise ValueError("weights from the chosen logits take no table, groups or correction")
+        self.router_bias = bool(p.get("router_bias", False))
+        if self.router_bias and self.weighting != "chosen":
+            raise ValueError("a router bias is served with weights from the chosen logits only")
+        self.clamp = p.get("clamp")
+        self.shared = p.get("shared")
+        self.shared_inter = int(self.shared["intermediate_size"]) if self.shared else 0
+        if self.clamp is None and self.shared:
+            raise ValueError("a shared expert is served beside clamped experts only")
+        if self.clamp is not None and not (float(self.clamp["limit"]) > 0
+                                           and (not self.shared or float(self.shared["limit"]) > 0)):
+            raise ValueError("a clamp must be positive")
+        self.width = self.experts * self.inter + self.shared_inter      # columns of the activations
+        self.router = self.correction = self.table = self.bias = None
         self.gate_up: Optional[Linear] = None
         self.down: Optional[Linear] = None
 
@@ -79,6 +107,12 @@ class RoutedFeedForward(Part):
             out = {n + "router": ParamSpec((self.E, self.hidden), role="gain", init="normal")}
         if self.correction_tensor and self.routing == "scores":
             out[n + "correction"] = ParamSpec((self.E,), role="gain", init="normal")
+        if self.router_bias:
+            out[n + "router.b"] = ParamSpec((self.E,), role="gain", init="normal")
+        if self.shared_inter:
+            out[n + "shared.gate"] = ParamSpec((self.shared_inter, self.hidden))
+            out[n + "shared.up"] = ParamSpec((self.shared_inter, self.hidden))
+            out[n + "shared.down"] = ParamSpec((self.hidden, self.shared_inter))
         for e in range(self.experts):
             out[f"{n}e{e}.gate"] = ParamSpec((self.inter, self.hidden))
             out[f"{n}e{e}.up"] = ParamSpec((self.inter, self.hidden))
@@ -95,6 +129,12 @@ class RoutedFeedForward(Part):
         else:
             self.router = tensors[n + "router"]              # float32: the router's product is never rounded
             self.correction = tensors[n + "correction"] if self.correction_tensor else None
+            self.bias = tensors[n + "router.b"] if self.router_bias else None
+        if self.clamp is not None:
+            names = [f"{n}e{e}." for e in range(self.experts)] + ([n + "shared."] if self.shared_inter else [])
+            self.gate_up = Linear(torch.cat([tensors[x + "gate"] for x in names] + [tensors[x + "up"] for x in names], dim=0))
+            self.down = Linear(torch.cat([tensors[x + "down"] for x in names], dim=1))
+            return
         rows = [torch.stack([tensors[f"{n}e{e}.gate"], tensors[f"{n}e{e}.up"]], dim=1).reshape(2 * F, d)
                 for e in range(self.experts)]
         self.gate_up = Linear(torch.cat(rows, dim=0))
@@ -116,19 +156,30 @@ class RoutedFeedForward(Part):
         weights = take("moe_weights", N, (self.E,), torch.float32)
         ids = take("moe_ids", N, (self.top,), torch.int32)
         picked = take("moe_picked", N, (self.top,), torch.float32)
+        if self.weighting == "chosen":
+            ops.moe_route_chosen(logits, self.bias, weights, ids, picked, self.top)
+            return weights, ids, picked
         ops.moe_route(logits, self.correction, weights, ids, picked, self.groups, self.keep, self.top)
         return weights, ids, picked
 
     def forward(self, ctx, x: torch.Tensor) -> Branch:
-        N, d, width = x.shape[0], self.hidden, self.experts * self.inter
+        N, d, width = x.shape[0], self.hidden, self.width
         weights, _, _ = self.route(ctx, x)
-        if ctx.can_fuse_silu_mul(N, self.gate_up.weight, x.dtype):
+        if self.clamp is not None:
+            gu = self.gate_up(ctx, x, "moe_gate_up", out="model_or_partial")
+            act = ctx.buffers.take("moe_act", N, (width,), ctx.dtype)
+            limit = float(self.clamp["limit"])
+            ops.moe_glu_clamp(act, gu, weights, self.experts, self.inter, limit,
+                              float(self.shared["limit"]) if self.shared else limit, float(self.clamp["alpha"]),
+                              float(self.clamp["offset"]))
+        elif ctx.can_fuse_silu_mul(N, self.gate_up.weight, x.dtype):
             act = self.gate_up(ctx, x, "moe_act", epilogue=1)
         else:
             gu = self.gate_up(ctx, x, "moe_gate_up")
             act = ctx.buffers.take("moe_act", N, (width,), ctx.dtype)
             ops.silu_mul(act, gu, interleaved=True)
-        ops.moe_scale(act, weights, self.experts)
+        if self.clamp is None:
+            ops.moe_scale(act, weights, self.experts)
         S = ctx.gemm_splits(N, self.down.weight, act.dtype)
         slabs = S + (1 if self.identity else 0)
         partial = ctx.buffers.take_flat("branch", slabs * N * d, torch.float32).view(slabs, N, d)
