@@ -474,6 +474,25 @@ def _magedra(width, heads):
             "streams": 4, "logit_scale": 1.0, "layers": four + again}
 
 
+def _samovik(width, heads):
+    """A Samovik configuration at real layer widths, eight layers: latent attention with heads of 128 + 32 dims over a
+    latent of 96 (a cached row of 128 dims) and a gate per head, two decayed linear attentions with a 128 x 128 state
+    per head, token-shift mixing with heads of 64, all twice; sixteen experts of half the width, four of them a
+    token, beside a shared one of twice the width (the products a token needs equal a dense gated feed-forward of
+    four times the width); a token input of an eighth of the width per layer."""
+    moe = {"kind": "moe", "expert": {"ff": width // 2, "limit": 7.0}, "router": {"experts": 16, "top": 4},
+           "shared": {"ff": 2 * width, "limit": 7.0}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {
+        "heads": heads, "dim": 128, "rot_dim": 32, "vdim": 128, "kv_rank": 96, "scale": 160 ** -0.5,
+        "rot": {"base": 1e4, "dims": 32, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    lin = {"type": "lightning", "mlp": moe, "mixer": {
+        "heads": heads, "dim": 128, "vdim": 128,
+        "decay": [1.0 - 2.0 ** (-2 - 8 * h / max(1, heads - 1)) for h in range(heads)]}}
+    wkv = {"type": "wkv", "mlp": moe, "mixer": {"heads": 2 * heads, "dim": 64}}
+    return {"architecture": "Samovik", "vocab": 32000, "width": width, "norm": {"eps": 1e-5},
+            "token_side": {"dim": width // 8}, "layers": [lat, lin, lin, wkv] * 2}
+
+
 def _qwen3_like(width, runs, heads):
     """The Qwen3 decoder at the same width, number of layer runs, head size and feed-forward width."""
     return {"architectures": ["Qwen3ForCausalLM"], "vocab_size": 32000, "hidden_size": width,
@@ -483,8 +502,9 @@ def _qwen3_like(width, runs, heads):
 
 
 def run_compare(args):
-    """`--compare bofusun|loletar|samerax|magedra`: prefill and decode throughput of another design at real layer widths
-    (random weights) beside the Qwen3 decoder at equal width, layer runs and head size.  One JSON line."""
+    """`--compare bofusun|loletar|samerax|magedra|samovik`: prefill and decode throughput of another design at real layer
+    widths (random weights) beside the Qwen3 decoder at equal width, layer runs and head size (Samovik: and beside
+    Loletar, whose layers carry routed experts and a matrix recurrence as well).  One JSON line."""
     import torch
 
     from socrates_b200 import Engine
@@ -506,10 +526,15 @@ def run_compare(args):
         width, heads = sizes[size]
         design = args.compare
         bof = {"bofusun": lambda: _bofusun(width, 5, heads, 1024), "loletar": lambda: _loletar(width, heads),
-               "samerax": lambda: _samerax(width, heads), "magedra": lambda: _magedra(width, heads)}[design]()
+               "samerax": lambda: _samerax(width, heads), "magedra": lambda: _magedra(width, heads),
+               "samovik": lambda: _samovik(width, heads)}[design]()
         runs = len(config_from_dict(bof).plan().order)
         only = [x for x in (args.only.split(",") if args.only else [design, "qwen3"])]
-        for label, cfg_dict in ((design, bof), ("qwen3", _qwen3_like(width, runs, heads))):
+        beside = [(design, bof), ("qwen3", _qwen3_like(width, runs, heads))]
+        if design == "samovik":
+            beside.insert(1, ("loletar", _loletar(width, heads)))
+            only = only if args.only else [design, "loletar", "qwen3"]
+        for label, cfg_dict in beside:
             if label not in only:
                 continue
             config = config_from_dict(cfg_dict)
@@ -630,7 +655,7 @@ def main():
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
-    ap.add_argument("--compare", default=None, choices=("bofusun", "loletar", "samerax", "magedra"),
+    ap.add_argument("--compare", default=None, choices=("bofusun", "loletar", "samerax", "magedra", "samovik"),
                     help="the Bofusun, the Loletar, the Samerax or the Magedra design at real layer widths beside Qwen3 at equal size "
                          "(prefill and decode); the default workload is not run")
     ap.add_argument("--only", default=None, help="with --compare: run only these of the pair, e.g. 'loletar' or 'qwen3'")

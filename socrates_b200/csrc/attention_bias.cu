@@ -24,7 +24,7 @@ namespace {
 constexpr int THREADS = 128;
 constexpr int KEYS = 128;      // keys per chunk: one per thread
 constexpr int HEADS = 4;       // query heads per pass over the keys
-constexpr int DMAX = 576;
+constexpr int DMAX = 640;
 
 struct BiasAttnArgs {
     void* out;                 // [N, Hq*Dv] in T
@@ -58,7 +58,8 @@ __device__ __forceinline__ float gate_factor(const BiasAttnArgs& a, int n, int h
     return 1.0f / (1.0f + expf(-z));
 }
 
-template <typename T>
+// NV: value dims a thread owns (thread t: dims t, t + THREADS, ...).
+template <typename T, int NV>
 __global__ void __launch_bounds__(THREADS) bias_attention_kernel(BiasAttnArgs a) {
     sb::pdl_launch_dependents();
     sb::pdl_wait();
@@ -90,9 +91,11 @@ __global__ void __launch_bounds__(THREADS) bias_attention_kernel(BiasAttnArgs a)
         // the sink is a key without a value: the first share of the keys starts from its term
         const bool sink_here = a.has_sink && blockIdx.z == 0;
         if (tid < HEADS) { run_max[tid] = sink_here ? a.sink : -INFINITY; run_sum[tid] = sink_here ? 1.f : 0.f; rescale[tid] = 0.f; }
-        float acc[HEADS][2];
+        float acc[HEADS][NV];
 #pragma unroll
-        for (int g = 0; g < HEADS; ++g) acc[g][0] = acc[g][1] = 0.f;
+        for (int g = 0; g < HEADS; ++g)
+#pragma unroll
+            for (int v = 0; v < NV; ++v) acc[g][v] = 0.f;
         __syncthreads();
         for (int c0 = lo; c0 < hi; c0 += KEYS) {
             const int nk = min(KEYS, hi - c0);
@@ -157,20 +160,23 @@ __global__ void __launch_bounds__(THREADS) bias_attention_kernel(BiasAttnArgs a)
                 }
             }
             __syncthreads();
-            // weighted sum of the values: thread t owns dims t and t + THREADS
+            // weighted sum of the values
 #pragma unroll
-            for (int g = 0; g < HEADS; ++g) { acc[g][0] *= rescale[g]; acc[g][1] *= rescale[g]; }
+            for (int g = 0; g < HEADS; ++g)
+#pragma unroll
+                for (int v = 0; v < NV; ++v) acc[g][v] *= rescale[g];
 #pragma unroll 8
             for (int t = 0; t < nk; ++t) {                      // the addresses come from shared memory: loads overlap
                 const int key = c0 + t;
                 const T* vr = vp + (((size_t)pg[t] * a.Hkv + kh) * BS + key % BS) * Dv;
-                const float v0 = tid < Dv ? to_float(vr[tid]) : 0.f;
-                const float v1 = tid + THREADS < Dv ? to_float(vr[tid + THREADS]) : 0.f;
+                float x[NV];
+#pragma unroll
+                for (int v = 0; v < NV; ++v) x[v] = tid + v * THREADS < Dv ? to_float(vr[tid + v * THREADS]) : 0.f;
 #pragma unroll
                 for (int g = 0; g < HEADS; ++g) {
                     if (g >= gn) continue;
-                    acc[g][0] = fmaf(w[g][t], v0, acc[g][0]);
-                    acc[g][1] = fmaf(w[g][t], v1, acc[g][1]);
+#pragma unroll
+                    for (int v = 0; v < NV; ++v) acc[g][v] = fmaf(w[g][t], x[v], acc[g][v]);
                 }
             }
             __syncthreads();
@@ -180,18 +186,21 @@ __global__ void __launch_bounds__(THREADS) bias_attention_kernel(BiasAttnArgs a)
             if (g >= gn) continue;
             const int h = h0 + g;
             // the gate scales the output, so it may scale every part
-            const float f0 = tid < Dv ? gate_factor<T>(a, n, h, tid) : 1.0f;
-            const float f1 = tid + THREADS < Dv ? gate_factor<T>(a, n, h, tid + THREADS) : 1.0f;
+            float f[NV];
+#pragma unroll
+            for (int v = 0; v < NV; ++v) f[v] = tid + v * THREADS < Dv ? gate_factor<T>(a, n, h, tid + v * THREADS) : 1.0f;
             if (a.NP == 1) {
-                const float f = 1.0f / run_sum[g];
+                const float inv = 1.0f / run_sum[g];
                 T* o = (T*)a.out + ((size_t)n * a.Hq + h) * Dv;
-                if (tid < Dv) o[tid] = from_float<T>(acc[g][0] * f * f0);
-                if (tid + THREADS < Dv) o[tid + THREADS] = from_float<T>(acc[g][1] * f * f1);
+#pragma unroll
+                for (int v = 0; v < NV; ++v)
+                    if (tid + v * THREADS < Dv) o[tid + v * THREADS] = from_float<T>(acc[g][v] * inv * f[v]);
             } else {
                 const size_t slot = ((size_t)n * a.Hq + h) * a.NP + blockIdx.z;
                 float* o = a.part_o + slot * Dv;
-                if (tid < Dv) o[tid] = acc[g][0] * f0;
-                if (tid + THREADS < Dv) o[tid + THREADS] = acc[g][1] * f1;
+#pragma unroll
+                for (int v = 0; v < NV; ++v)
+                    if (tid + v * THREADS < Dv) o[tid + v * THREADS] = acc[g][v] * f[v];
                 if (tid == 0) {                          // an empty part has sum 0 and is skipped by the merge
                     a.part_ml[slot * 2] = run_max[g];
                     a.part_ml[slot * 2 + 1] = run_sum[g];
@@ -371,8 +380,8 @@ extern "C" int sb_attention_bias(void* out, const void* q, const void* k_pool, c
                                  float sink, cudaStream_t stream) {
     SB_REQUIRE(N >= 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0,
                "attention_bias: %d query heads are no multiple of %d KV heads", Hq, Hkv);
-    SB_REQUIRE(Dk >= 1 && Dk <= DMAX && Dv >= 1 && Dv <= 2 * THREADS,
-               "attention_bias: head sizes %d (keys) and %d (values) must be at most %d", Dk, Dv, DMAX);
+    SB_REQUIRE(Dk >= 1 && Dk <= DMAX && Dv >= 1 && Dv <= 4 * THREADS,
+               "attention_bias: head sizes %d (keys, at most %d) and %d (values, at most %d)", Dk, DMAX, Dv, 4 * THREADS);
     SB_REQUIRE(page_size > 0 && table_width > 0, "attention_bias: bad page_size %d or table width %d", page_size,
                table_width);
     SB_REQUIRE(window >= 0, "attention_bias: window %d is negative", window);
@@ -391,12 +400,14 @@ extern "C" int sb_attention_bias(void* out, const void* q, const void* k_pool, c
     a.gate_per_dim = gate_per_dim; a.has_sink = has_sink; a.sink = sink;
     dim3 grid(Hkv, N, num_partitions), rgrid(Hq, N);
     if (dtype == SB_F32) {
-        sb::launch(bias_attention_kernel<float>, grid, dim3(THREADS), 0, stream, a);
+        if (Dv > 2 * THREADS) sb::launch(bias_attention_kernel<float, 4>, grid, dim3(THREADS), 0, stream, a);
+        else sb::launch(bias_attention_kernel<float, 2>, grid, dim3(THREADS), 0, stream, a);
         if (num_partitions > 1)
             sb::launch(attn_reduce_kernel<float>, rgrid, dim3(128), 0, stream, (float*)out, (const float*)part_o,
                        (const float*)part_ml, Hq, Dv, num_partitions);
     } else if (dtype == SB_BF16) {
-        sb::launch(bias_attention_kernel<__nv_bfloat16>, grid, dim3(THREADS), 0, stream, a);
+        if (Dv > 2 * THREADS) sb::launch(bias_attention_kernel<__nv_bfloat16, 4>, grid, dim3(THREADS), 0, stream, a);
+        else sb::launch(bias_attention_kernel<__nv_bfloat16, 2>, grid, dim3(THREADS), 0, stream, a);
         if (num_partitions > 1)
             sb::launch(attn_reduce_kernel<__nv_bfloat16>, rgrid, dim3(128), 0, stream, (__nv_bfloat16*)out,
                        (const float*)part_o, (const float*)part_ml, Hq, Dv, num_partitions);

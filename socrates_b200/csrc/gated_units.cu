@@ -215,6 +215,146 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(HeadArgs a) {
     }
 }
 
+// The same for up to 16 tokens (decode steps): 32 outputs a block, eight threads an output, each with every eighth
+// run of eight inputs, so that a head's matrix is one round trip to memory; their shares are joined in a fixed order.
+template <typename T>
+__global__ void __launch_bounds__(256) head_matmul_few_kernel(HeadArgs a) {
+    sb::pdl_launch_dependents();
+    extern __shared__ __align__(16) float few[];             // x [HT][nin rounded up to 64], then the shares [8][32][HT + 1]
+    const int h = blockIdx.x, o = blockIdx.z * 32 + (threadIdx.x & 31), ks = threadIdx.x >> 5;
+    const int nin = a.transposed ? a.A : a.B, nout = a.transposed ? a.B : a.A, np = (nin + 63) & ~63;
+    float* xs = few;
+    float* sh = xs + HT * np;
+    const T* w = (const T*)a.w + (size_t)h * a.A * a.B;
+    sb::pdl_wait();
+    const T* x = (const T*)a.x + a.x_off + (size_t)h * a.x_head;
+    T* y = (T*)a.y + a.y_off + (size_t)h * a.y_head;
+    if (blockIdx.z == 0 && a.carry > 0) {
+        for (int i = threadIdx.x; i < a.N * a.carry; i += 256) {
+            const int t = i / a.carry, c = i - t * a.carry;
+            y[(size_t)t * a.y_stride - a.carry + c] = x[(size_t)t * a.x_stride - a.carry + c];
+        }
+    }
+    for (int i = threadIdx.x; i < HT * np; i += 256) {
+        const int t = i / np, d = i - t * np;
+        xs[i] = t < a.N && d < nin ? to_float(x[(size_t)t * a.x_stride + d]) : 0.f;
+    }
+    __syncthreads();
+    float acc[HT];
+#pragma unroll
+    for (int t = 0; t < HT; ++t) acc[t] = 0.f;
+    if (o < nout) {
+        for (int d0 = ks * 8; d0 < nin; d0 += 64) {
+            float wv[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                wv[e] = 0.f;
+                if (d0 + e < nin) wv[e] = to_float(a.transposed ? w[(size_t)(d0 + e) * a.B + o] : w[(size_t)o * a.B + d0 + e]);
+            }
+#pragma unroll
+            for (int t = 0; t < HT; ++t)
+                if (t < a.N) {
+#pragma unroll
+                    for (int e = 0; e < 8; e += 4) {
+                        const float4 v = *reinterpret_cast<const float4*>(xs + t * np + d0 + e);
+                        acc[t] = fmaf(wv[e], v.x, fmaf(wv[e + 1], v.y, fmaf(wv[e + 2], v.z, fmaf(wv[e + 3], v.w, acc[t]))));
+                    }
+                }
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < HT; ++t) sh[(ks * 32 + (threadIdx.x & 31)) * (HT + 1) + t] = acc[t];
+    __syncthreads();
+    for (int i = threadIdx.x; i < 32 * a.N; i += 256) {
+        const int t = i / 32, oo = i - t * 32;
+        if (blockIdx.z * 32 + oo >= nout) continue;
+        float v = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += sh[(k * 32 + oo) * (HT + 1) + t];
+        y[(size_t)t * a.y_stride + blockIdx.z * 32 + oo] = from_float<T>(v);
+    }
+}
+
+// The same on mma.sync (bfloat16, float32 accumulation) for prompt portions: 64 tokens x 64 outputs a block, the
+// inputs in steps of 64.
+constexpr int HM = 64, HLD = HM + 8;
+
+__device__ __forceinline__ uint32_t shared_address(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
+
+__global__ void __launch_bounds__(128) head_matmul_mma_kernel(HeadArgs a) {
+    sb::pdl_launch_dependents();
+    typedef __nv_bfloat16 bf;
+    __shared__ __align__(16) bf xs[HM][HLD], wsm[HM][HLD];
+    const int h = blockIdx.x, n0 = blockIdx.y * HM, o0 = blockIdx.z * HM, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int nin = a.transposed ? a.A : a.B, nout = a.transposed ? a.B : a.A;
+    const bf* w = (const bf*)a.w + (size_t)h * a.A * a.B;
+    sb::pdl_wait();
+    const bf* x = (const bf*)a.x + a.x_off + (size_t)h * a.x_head;
+    bf* y = (bf*)a.y + a.y_off + (size_t)h * a.y_head;
+    const int nt = min(HM, a.N - n0);
+    if (blockIdx.z == 0 && a.carry > 0) {
+        for (int i = tid; i < nt * a.carry; i += 128) {
+            const int t = i / a.carry, c = i - t * a.carry;
+            y[(size_t)(n0 + t) * a.y_stride - a.carry + c] = x[(size_t)(n0 + t) * a.x_stride - a.carry + c];
+        }
+    }
+    float acc[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    for (int k0 = 0; k0 < nin; k0 += HM) {
+        __syncthreads();
+#pragma unroll
+        for (int i = tid; i < HM * HM / 8; i += 128) {
+            const int r = i / (HM / 8), c = (i - r * (HM / 8)) * 8;
+            uint4 v = make_uint4(0u, 0u, 0u, 0u), u = v;
+            if (r < nt && k0 + c < nin) v = *reinterpret_cast<const uint4*>(x + (size_t)(n0 + r) * a.x_stride + k0 + c);
+            // rows of the staged matrix: outputs (columns: inputs), or, transposed, inputs (columns: outputs)
+            if (a.transposed ? (k0 + r < nin && o0 + c < nout) : (o0 + r < nout && k0 + c < nin))
+                u = *reinterpret_cast<const uint4*>(w + (a.transposed ? (size_t)(k0 + r) * a.B + o0 + c : (size_t)(o0 + r) * a.B + k0 + c));
+            *reinterpret_cast<uint4*>(&xs[r][c]) = v;
+            *reinterpret_cast<uint4*>(&wsm[r][c]) = u;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int kk = 0; kk < HM; kk += 16) {
+            uint32_t q[4];
+            const uint32_t qa = shared_address(&xs[warp * 16 + (lane & 15)][kk + (lane >> 4) * 8]);
+            asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                         : "=r"(q[0]), "=r"(q[1]), "=r"(q[2]), "=r"(q[3]) : "r"(qa));
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {                  // two groups of eight outputs a load
+                uint32_t b[4];
+                if (a.transposed) {
+                    const uint32_t ba = shared_address(&wsm[kk + (lane & 15)][j * 8 + (lane >> 4) * 8]);
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+                                 : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(ba));
+                } else {
+                    const uint32_t ba = shared_address(&wsm[j * 8 + (lane & 7) + ((lane >> 4) << 3)][kk + ((lane >> 3) & 1) * 8]);
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                                 : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(ba));
+                }
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    asm volatile(
+                        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+                        "{%0, %1, %2, %3};"
+                        : "+f"(acc[j + e][0]), "+f"(acc[j + e][1]), "+f"(acc[j + e][2]), "+f"(acc[j + e][3])
+                        : "r"(q[0]), "r"(q[1]), "r"(q[2]), "r"(q[3]), "r"(b[2 * e]), "r"(b[2 * e + 1]));
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int t = warp * 16 + (lane >> 2) + 8 * e, o = o0 + j * 8 + (lane & 3) * 2;
+            if (t < nt && o < nout) {
+                __nv_bfloat162 v = __floats2bfloat162_rn(acc[j][2 * e], acc[j][2 * e + 1]);
+                *reinterpret_cast<__nv_bfloat162*>(y + (size_t)(n0 + t) * a.y_stride + o) = v;
+            }
+        }
+}
+
 struct LatentArgs {
     const void* down;          // [N, stride] in T: the latent at c_off (rank), the shared key part at r_off (dr)
     long long stride;
@@ -373,7 +513,23 @@ extern "C" int sb_head_matmul(void* y, long long y_stride, int y_off, int y_head
     HeadArgs a;
     a.x = x; a.x_stride = x_stride; a.x_off = x_off; a.x_head = x_head; a.y = y; a.y_stride = y_stride;
     a.y_off = y_off; a.y_head = y_head; a.w = w; a.A = A; a.B = B; a.transposed = transposed; a.carry = carry; a.N = N;
-    const int nout = transposed ? B : A;
+    const int nout = transposed ? B : A, nin = transposed ? A : B;
+    const size_t few = ((size_t)HT * ((nin + 63) & ~63) + 8 * 32 * (HT + 1)) * sizeof(float);
+    if (N <= HT && few <= 48 * 1024 && (nout + 31) / 32 <= 65535) {
+        const dim3 fgrid(H, 1, (nout + 31) / 32);
+        if (dtype == SB_F32) sb::launch(head_matmul_few_kernel<float>, fgrid, dim3(256), few, stream, a);
+        else if (dtype == SB_BF16) sb::launch(head_matmul_few_kernel<__nv_bfloat16>, fgrid, dim3(256), few, stream, a);
+        else SB_REQUIRE(false, "head_matmul: unknown dtype %d", dtype);
+        SB_LAUNCH_CHECK();
+    }
+    // 16-byte pieces of every row (inputs and matrix) and 4-byte pieces of the outputs
+    const bool pieces = nin % 8 == 0 && nout % 8 == 0 && x_stride % 8 == 0 && x_off % 8 == 0 && x_head % 8 == 0 &&
+                        ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0 &&
+                        (reinterpret_cast<uintptr_t>(y) & 3) == 0 && y_stride % 2 == 0 && y_off % 2 == 0 && y_head % 2 == 0;
+    if (dtype == SB_BF16 && pieces && N > 32 && (N + HM - 1) / HM <= 65535) {
+        sb::launch(head_matmul_mma_kernel, dim3(H, (N + HM - 1) / HM, (nout + HM - 1) / HM), dim3(128), 0, stream, a);
+        SB_LAUNCH_CHECK();
+    }
     const dim3 grid(H, (N + HT - 1) / HT, (nout + 127) / 128);
     SB_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "head_matmul: %d tokens exceed one launch", N);
     if (dtype == SB_F32) sb::launch(head_matmul_kernel<float>, grid, dim3(128), 0, stream, a);

@@ -7,7 +7,8 @@
 //                largest c; only the `keep` best groups stay (the others' c count as -inf)
 //                the `top` largest c are chosen; their weights are s (no correction, not renormalized)
 //                weights[n][e] = s_e for chosen e, else 0 ;  ids[n][k], picked[n][k] = the choices, best first
-//   route, chosen: the `top` largest of z + bias are chosen; their weights are the softmax over these only
+//   router:      logits and choice in one kernel: the `top` largest of z + bias are chosen; their weights are the
+//                softmax over these only
 //   glu_clamp:   all experts' gated units and the shared one's in one pass, scaled on the way out:
 //                g = min(pg, limit) ,  u = clamp(pu, -limit, limit) ,  act = g * sigmoid(alpha g) * (u + offset) * weight
 //   scale:       act[n][e*F + f] *= weights[n][e]                (all experts' activations side by side)
@@ -113,46 +114,120 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(
     }
 }
 
-// Weights from the chosen logits only: a warp per token, ties to the lower index.
-__global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_chosen_kernel(
-    const float* __restrict__ logits, const float* __restrict__ bias, float* __restrict__ weights, int* __restrict__ ids,
-    float* __restrict__ picked, int N, int E, int top) {
+// The router's product and the choice by its logits in one kernel, TT tokens a block.  A warp makes an
+// output's logits for all of them: lane l takes elements 4 l .. 4 l + 3 of every 128, in order, one sum a lane joined in a fixed
+// tree, so a token's logits do not depend on what else the step holds.  Then a warp per token picks the `top` largest
+// of logit + bias (ties to the lower index) and writes the softmax over these.
+struct RouterArgs {
+    const void* x;             // [N, K] in T
+    const float* router;       // [E, K]
+    const float* bias;         // [E] or null
+    float* weights;            // [N, E]
+    int* ids;                  // [N, top]
+    float* picked;             // [N, top]
+    int N, E, K, top;
+};
+
+template <typename T, int TT>
+__global__ void __launch_bounds__(TT == 1 ? 1024 : 256) moe_router_kernel(RouterArgs a) {
     sb::pdl_launch_dependents();
-    extern __shared__ float rsm[];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    float* c = rsm + (size_t)warp * 2 * E;                  // open logits
-    float* w = c + E;                                       // weights
-    const int n = blockIdx.x * ROUTE_WARPS + warp;
+    extern __shared__ __align__(16) float rsm[];
+    const int K = a.K, E = a.E, Kp = (K + 127) / 128 * 128;
+    float* xs = rsm;                                         // [TT][Kp]
+    float* zs = xs + TT * Kp;                                // [TT][2 E]: open logits, weights
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n0 = blockIdx.x * TT, warps = blockDim.x >> 5;
     sb::pdl_wait();
-    if (n >= N) return;
-    for (int e = lane; e < E; e += 32) {
-        c[e] = logits[(size_t)n * E + e] + (bias ? bias[e] : 0.f);
-        w[e] = 0.f;
-    }
-    __syncwarp();
-    float best = 0.f, sum = 0.f;
-    for (int k = 0; k < top; ++k) {
-        float bv = -INFINITY;
-        int bi = 0x7fffffff;
-        for (int e = lane; e < E; e += 32) {
-            const float v = c[e];
-            if (!isnan(v) && (v > bv || (bi == 0x7fffffff && w[e] == 0.f))) { bv = v; bi = e; }
+    const T* x = (const T*)a.x;
+    constexpr int VEC = Vec16<T>::N;
+    if (K % VEC == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+        for (int i = threadIdx.x * VEC; i < TT * Kp; i += blockDim.x * VEC) {
+            const int t = i / Kp, k = i - t * Kp;
+            Vec16<T> v;
+            const bool have = n0 + t < a.N && k < K;
+            if (have) v.load(x + (size_t)(n0 + t) * K + k);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) xs[i + e] = have ? v.get(e) : 0.f;
         }
-        warp_argmax(bv, bi);
-        if (k == 0) best = bv;
-        const float p = expf(bv - best);
-        sum += p;
-        if (lane == 0 && bi < E) {
-            ids[(size_t)n * top + k] = bi;
-            picked[(size_t)n * top + k] = p;
-            w[bi] = p;
-            c[bi] = NAN;                                     // taken
+    } else {
+        for (int i = threadIdx.x; i < TT * Kp; i += blockDim.x) {
+            const int t = i / Kp, k = i - t * Kp;
+            xs[i] = n0 + t < a.N && k < K ? to_float(x[(size_t)(n0 + t) * K + k]) : 0.f;
         }
-        __syncwarp();
     }
-    const float inv = 1.0f / sum;
-    for (int e = lane; e < E; e += 32) weights[(size_t)n * E + e] = w[e] * inv;
-    for (int k = lane; k < top; k += 32) picked[(size_t)n * top + k] *= inv;
+    __syncthreads();
+    const bool wide = K % 4 == 0;
+    for (int e = warp; e < E; e += warps) {
+        const float* w = a.router + (size_t)e * K;
+        float acc[TT];
+#pragma unroll
+        for (int t = 0; t < TT; ++t) acc[t] = 0.f;
+#pragma unroll (TT == 1 ? 8 : 4)
+        for (int k = lane * 4; k < Kp; k += 128) {
+            float4 wv = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (wide) {
+                if (k < K) wv = __ldg(reinterpret_cast<const float4*>(w + k));
+            } else {
+                if (k < K) wv.x = w[k];
+                if (k + 1 < K) wv.y = w[k + 1];
+                if (k + 2 < K) wv.z = w[k + 2];
+                if (k + 3 < K) wv.w = w[k + 3];
+            }
+#pragma unroll
+            for (int t = 0; t < TT; ++t) {
+                const float4 xv = *reinterpret_cast<const float4*>(xs + t * Kp + k);
+                acc[t] = fmaf(xv.x, wv.x, fmaf(xv.y, wv.y, fmaf(xv.z, wv.z, fmaf(xv.w, wv.w, acc[t]))));
+            }
+        }
+        const float b = a.bias ? a.bias[e] : 0.f;
+#pragma unroll
+        for (int t = 0; t < TT; ++t) {
+            const float z = warp_sum(acc[t]);
+            if (lane == 0) {
+                zs[t * 2 * E + e] = z + b;
+                zs[t * 2 * E + E + e] = 0.f;
+            }
+        }
+    }
+    __syncthreads();
+    for (int t = warp; t < TT; t += warps) {
+        const int n = n0 + t;
+        if (n >= a.N) break;
+        float *c = zs + t * 2 * E, *w = c + E;
+        float best = 0.f, sum = 0.f;
+        for (int k = 0; k < a.top; ++k) {
+            float bv = -INFINITY;
+            int bi = 0x7fffffff;
+            for (int e = lane; e < E; e += 32) {
+                const float v = c[e];
+                if (!isnan(v) && (v > bv || bi == 0x7fffffff)) { bv = v; bi = e; }
+            }
+            warp_argmax(bv, bi);
+            if (k == 0) best = bv;
+            const float p = expf(bv - best);
+            sum += p;
+            if (lane == 0 && bi < E) {
+                a.ids[(size_t)n * a.top + k] = bi;
+                w[bi] = p;
+                c[bi] = NAN;                                 // taken
+            }
+            __syncwarp();
+        }
+        const float inv = 1.0f / sum;
+        for (int e = lane; e < E; e += 32) a.weights[(size_t)n * E + e] = w[e] * inv;
+        for (int k = lane; k < a.top; k += 32) a.picked[(size_t)n * a.top + k] = w[a.ids[(size_t)n * a.top + k]] * inv;
+    }
+}
+
+template <typename T, int TT>
+void launch_router(const RouterArgs& a, size_t smem, cudaStream_t stream) {
+    static sb::OncePerDevice once;
+    if (smem > 48 * 1024 && !once.flag()) {
+        cudaFuncSetAttribute(moe_router_kernel<T, TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        once.flag() = true;
+    }
+    // one token: a warp per output as far as a block goes, so that its rows are on their way together
+    const int warps = TT > 1 ? 8 : a.E < 8 ? 8 : a.E > 32 ? 32 : a.E;
+    sb::launch(moe_router_kernel<T, TT>, dim3((a.N + TT - 1) / TT), dim3(32 * warps), smem, stream, a);
 }
 
 // Column f < experts * F belongs to expert f / F; the columns from there on to the shared expert, whose weight is
@@ -385,14 +460,21 @@ extern "C" int sb_moe_route(const float* logits, const float* correction, float*
     SB_LAUNCH_CHECK();
 }
 
-extern "C" int sb_moe_route_chosen(const float* logits, const float* bias, float* weights, int* ids, float* picked, int N,
-                                   int E, int top, cudaStream_t stream) {
-    SB_REQUIRE(N >= 0 && E > 0 && top >= 1 && top <= E, "moe_route_chosen: bad sizes N=%d E=%d top=%d", N, E, top);
-    const size_t smem = (size_t)ROUTE_WARPS * 2 * E * sizeof(float);
-    SB_REQUIRE(smem <= 48 * 1024, "moe_route_chosen: %d router outputs do not fit a block's shared memory", E);
+// weights float32 [N, E]; ids int32 and picked float32 [N, top].
+extern "C" int sb_moe_router(const void* x, const float* router, const float* bias, float* weights, int* ids, float* picked,
+                             int N, int E, int K, int top, int dtype, cudaStream_t stream) {
+    SB_REQUIRE(N >= 0 && E > 0 && K > 0 && top >= 1 && top <= E, "moe_router: bad sizes N=%d E=%d K=%d top=%d", N, E, K, top);
+    const int Kp = (K + 127) / 128 * 128;
+    auto need = [&](int tt) { return (size_t)tt * (Kp + 2 * E) * sizeof(float); };
+    SB_REQUIRE(need(1) <= 200 * 1024, "moe_router: rows of %d values and %d outputs do not fit a block's shared memory", K, E);
+    SB_REQUIRE(dtype == SB_F32 || dtype == SB_BF16, "moe_router: unknown dtype %d", dtype);
     if (N == 0) return 0;
-    sb::launch(moe_route_chosen_kernel, dim3((N + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, stream,
-               logits, bias, weights, ids, picked, N, E, top);
+    RouterArgs a;
+    a.x = x; a.router = router; a.bias = bias; a.weights = weights; a.ids = ids; a.picked = picked; a.N = N; a.E = E; a.K = K;
+    a.top = top;
+    const bool many = N >= 512 && need(8) <= 100 * 1024;      // many tokens: a router row fetched once serves eight
+    if (dtype == SB_F32) { if (many) launch_router<float, 8>(a, need(8), stream); else launch_router<float, 1>(a, need(1), stream); }
+    else { if (many) launch_router<__nv_bfloat16, 8>(a, need(8), stream); else launch_router<__nv_bfloat16, 1>(a, need(1), stream); }
     SB_LAUNCH_CHECK();
 }
 

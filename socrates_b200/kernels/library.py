@@ -82,7 +82,9 @@ _SIGNATURES = {
     "sb_linear_recurrence": [P] + [P, I, LL, LL, I] * 4 + [P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, P, P, I, P],
     "sb_norm_gate": [P, P, P, I, LL, LL, I, P, I, I, I, F, I, I, P],
     "sb_token_shift_mix": [P, P, P, P, P, I, I, I, I, P],
-    "sb_moe_route_chosen": [P, P, P, P, P, I, I, I, P],
+    "sb_moe_router": [P, P, P, P, P, P, I, I, I, I, I, P],
+    "sb_attention_latent_supports": [I, I, I],
+    "sb_attention_latent": [P, P, P, P, I, P, P, P, P, P, I, P, LL, I, I, I, I, I, I, F, I, I, P, P, P],
     "sb_moe_glu_clamp": [P, P, P, I, LL, P, I, I, I, I, I, F, F, F, F, I, P],
     "sb_segment_norm": [P, LL, I, P, P, P, P, P, P, P, P, P, F, I, I, P],
     "sb_head_matmul": [P, LL, I, I, P, LL, I, I, P, I, I, I, I, I, I, I, P],

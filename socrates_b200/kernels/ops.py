@@ -1531,20 +1531,23 @@ def token_shift_mix(out: torch.Tensor, x: torch.Tensor, mu: torch.Tensor, last: 
                                       _code(x.dtype), _stream()), "token_shift_mix")
 
 
-def moe_route_chosen(logits: torch.Tensor, bias: Optional[torch.Tensor], weights: torch.Tensor, ids: torch.Tensor,
-                     picked: torch.Tensor, top: int) -> None:
-    """Choose the `top` largest of logits + bias per token; weights float32 [N, E] gets the softmax over the chosen
-    ones at their places and 0 elsewhere, ids int32 / picked float32 [N, top] the choices best first."""
-    N, E = logits.shape
-    _want(logits, "logits", torch.float32)
+def moe_router(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], weights: torch.Tensor,
+               ids: torch.Tensor, picked: torch.Tensor, top: int) -> None:
+    """Logits z = x [N, K] @ router [E, K]^T + bias (float32 weights and sums, made in the same order whatever else the
+    step holds) and the choice by them: weights float32 [N, E] gets the softmax over the `top` largest logits at their
+    places and 0 elsewhere, ids int32 / picked float32 [N, top] the choices best first."""
+    N, K = x.shape
+    E = router.shape[0]
+    _want(x, "x")
+    _want(router, "router", torch.float32, (E, K))
     if bias is not None:
         _want(bias, "bias", torch.float32, (E,))
     _want(weights, "weights", torch.float32, (N, E))
     _want(ids, "ids", torch.int32, (N, top))
     _want(picked, "picked", torch.float32, (N, top))
     lib = library()
-    check(lib, lib.sb_moe_route_chosen(_ptr(logits), _ptr(bias), _ptr(weights), _ptr(ids), _ptr(picked), N, E, int(top),
-                                       _stream()), "moe_route_chosen")
+    check(lib, lib.sb_moe_router(_ptr(x), _ptr(router), _ptr(bias), _ptr(weights), _ptr(ids), _ptr(picked), N, E, K,
+                                 int(top), _code(x.dtype), _stream()), "moe_router")
 
 
 def moe_glu_clamp(out: torch.Tensor, x: torch.Tensor, weights: torch.Tensor, experts: int, inter: int, limit: float,
@@ -1588,3 +1591,46 @@ def gelu_lookup(out: torch.Tensor, x: torch.Tensor, table: torch.Tensor, first: 
     check(lib, lib.sb_gelu_lookup(_ptr(out), None if parts else _ptr(x), _ptr(x) if parts else None,
                                   x.shape[0] if parts else 0, N * F_, _ptr(table), table.stride(0), int(first), _ptr(ids),
                                   _ptr(feedback), table.shape[0], N, F_, _code(out.dtype), _stream()), "gelu_lookup")
+
+
+def attention_latent_supports(num_heads: int, row_dim: int, latent_dim: int) -> bool:
+    """Whether the tensor-core kernel over one cached head takes rows of this size (bfloat16, multiples of 8)."""
+    return bool(library().sb_attention_latent_supports(int(num_heads), int(row_dim), int(latent_dim)))
+
+
+def attention_latent(out: torch.Tensor, q: torch.Tensor, pool: torch.Tensor, rank: int, block_table: torch.Tensor,
+                     token_rows: torch.Tensor, positions: torch.Tensor, seq_starts: torch.Tensor, seq_rows: torch.Tensor,
+                     seq_first_pos: torch.Tensor, num_heads: int, scale: float, window: int = 0,
+                     gate: Optional[torch.Tensor] = None, prompt: bool = False, num_partitions: int = 1,
+                     part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None) -> None:
+    """Paged causal attention of all heads over ONE cached head (bfloat16): q [N, H*D], pool [pages, 1, BS, D], whose
+    rows are the keys and whose last `rank` dims are the values; out [N, H*rank], times sigmoid(gate[:, h]) where a gate
+    [N, >= H] is given.  Scores, softmax and sums are float32, both products run on the tensor cores and each softmax
+    weight enters the second as two bfloat16 terms.  `prompt`: tiles of consecutive tokens of a request; otherwise every
+    token is a tile and its keys are cut into `num_partitions` shares (scratch as `attention_bias`)."""
+    N, H = q.shape[0], num_heads
+    pages, heads, BS, D = pool.shape
+    R = seq_rows.numel()
+    _want(q, "q", torch.bfloat16, (N, H * D))
+    _want(pool, "pool", torch.bfloat16, (pages, 1, BS, D))
+    _want(out, "out", torch.bfloat16, (N, H * rank))
+    _want(block_table, "block_table", torch.int32)
+    _want(token_rows, "token_rows", torch.int32, (N,))
+    _want(positions, "positions", torch.int32, (N,))
+    _want(seq_starts, "seq_starts", torch.int32, (R + 1,))
+    _want(seq_rows, "seq_rows", torch.int32, (R,))
+    _want(seq_first_pos, "seq_first_pos", torch.int32, (R,))
+    gate_stride = _gate_stride(gate, q, N, H)
+    NP = 1 if prompt else int(num_partitions)
+    if NP > 1:
+        _want(part_o, "part_o", torch.float32)
+        _want(part_ml, "part_ml", torch.float32)
+        if part_o.numel() < N * H * NP * rank or part_ml.numel() < N * H * NP * 2:
+            raise KernelError("attention scratch buffers are too small")
+    lib = library()
+    check(lib, lib.sb_attention_latent(_ptr(out), _ptr(q), _ptr(pool), _ptr(block_table), block_table.shape[1],
+                                       _ptr(token_rows), _ptr(positions), _ptr(seq_starts), _ptr(seq_rows),
+                                       _ptr(seq_first_pos), R, _ptr(gate), gate_stride, N, H, D, int(rank), BS, int(window),
+                                       float(scale), int(bool(prompt)), NP, _ptr(part_o) if NP > 1 else None,
+                                       _ptr(part_ml) if NP > 1 else None, _stream()), "attention_latent",
+          kernels=2 if NP > 1 else 1)

@@ -17,8 +17,9 @@ when the weights are bound so that every head's turning part comes first; withou
 latent, the key part and the gate are one product.  One kernel norms the latent, turns
 the key part and the queries and writes the token's row into its pages.
 Norms, angles, scores, weights and sums are float32; the per-head matrices accumulate in float32.  One exception, in
-the bfloat16 engine only: prompt portions of layers whose cached row has 64 or 128 dims run on the tensor-core tile
-kernel (the key rows serve as values too), where each softmax weight enters the value product as two bfloat16 terms.
+the bfloat16 engine only: attention runs on the tensor cores (prompt portions of layers whose cached row has 64 or 128
+dims on the tile kernel, the key rows serving as values too; everything else on a kernel of its own for one cached
+head, where the row's sizes are multiples of 8), and each softmax weight enters the value product as two bfloat16 terms.
 Tensors: `<name>dq`, `dq.norm`, `uq` (or `q`), `dkv`, `dkv.norm`, `uk`, `uv`, `g`, `o`.
 """
 
@@ -53,9 +54,9 @@ class LatentAttention(Part):
         self.D = self.dr + self.kv_rank                  # the cached key row: [k_rot | c]
         if self.dr % 2:
             raise ValueError(f"{self.dr} turning dims are not even")
-        if not (1 <= self.D <= 576 and self.kv_rank <= 256):
-            raise ValueError(f"a cached row of {self.dr} + {self.kv_rank} dims; the kernels take up to 576, with a "
-                             f"latent of up to 256")
+        if not (1 <= self.D <= 640 and self.kv_rank <= 512):
+            raise ValueError(f"a cached row of {self.dr} + {self.kv_rank} dims; the kernels take up to 640, with a "
+                             f"latent of up to 512")
         self.down: Optional[Linear] = None
         self.uq: Optional[Linear] = None
         self.o: Optional[Linear] = None
@@ -109,7 +110,11 @@ class LatentAttention(Part):
 
     def forward(self, ctx, x: torch.Tensor, cache) -> Branch:
         N, H, D, rank, dr, dn = x.shape[0], self.H, self.D, self.kv_rank, self.dr, self.dn
-        down = self.down(ctx, x, "la_down")                                  # [c_q raw or q | c raw | k_rot raw | gate]
+        # [c_q raw or q | c raw | k_rot raw | gate]; a decode step cuts the product along K and adds the parts
+        down = self.down(ctx, x, "la_down_parts", out="model_or_partial")
+        if down.dim() == 3:
+            parts, down = down, ctx.buffers.take("la_down", N, (self.down.out_features,), ctx.dtype)
+            ops.bias_act(down, parts, None, "identity")
         c_off = self.c_off
         gate = down[:, c_off + rank + dr:] if self.gated else None
         if self.q_rank:
@@ -139,6 +144,16 @@ class LatentAttention(Part):
             ops.attention_prefill_tcgen05(src, q, k_pool, k_pool, table, ctx.seq_starts, ctx.seq_rows, ctx.seq_first_pos,
                                           H, self.scale, ctx.status, self.window or 0, gate=gate)
             first, step = dr, D
+        elif ctx.dtype == torch.bfloat16 and ops.attention_latent_supports(H, D, rank):
+            # every other step of the bfloat16 engine: both products on mma.sync, the cached rows read once
+            src = ctx.buffers.take("la_lat", N, (H * rank,), ctx.dtype)
+            prompt = not ctx.all_decode and N >= 4 * ctx.num_seqs
+            NP, part_o, part_ml = 1 if prompt else self.partitions(ctx, N, cache.manager.max_len), None, None
+            if NP > 1:
+                part_o = ctx.buffers.take_flat("attn_part_o", N * H * NP * rank, torch.float32)
+                part_ml = ctx.buffers.take_flat("attn_part_ml", N * H * NP * 2, torch.float32)
+            ops.attention_latent(src, q, k_pool, rank, table, ctx.token_rows, ctx.positions, ctx.seq_starts, ctx.seq_rows,
+                                 ctx.seq_first_pos, H, self.scale, self.window or 0, gate, prompt, NP, part_o, part_ml)
         elif (not ctx.all_decode and N >= 4 * ctx.num_seqs
                 and ops.attention_bias_tile_supports(H, 1, D, rank, ctx.dtype)):
             src = ctx.buffers.take("la_lat", N, (H * rank,), ctx.dtype)

@@ -151,14 +151,14 @@ class RoutedFeedForward(Part):
             weights = take("moe_weights", N, (self.E,), torch.float32)
             ops.moe_table(weights, ctx.token_ids, self.table, ctx.token_feedback)
             return weights, None, None
-        logits = take("moe_logits", N, (self.E,), torch.float32)
-        ops.moe_logits(logits, x, self.router)
         weights = take("moe_weights", N, (self.E,), torch.float32)
         ids = take("moe_ids", N, (self.top,), torch.int32)
         picked = take("moe_picked", N, (self.top,), torch.float32)
         if self.weighting == "chosen":
-            ops.moe_route_chosen(logits, self.bias, weights, ids, picked, self.top)
+            ops.moe_router(x, self.router, self.bias, weights, ids, picked, self.top)
             return weights, ids, picked
+        logits = take("moe_logits", N, (self.E,), torch.float32)
+        ops.moe_logits(logits, x, self.router)
         ops.moe_route(logits, self.correction, weights, ids, picked, self.groups, self.keep, self.top)
         return weights, ids, picked
 
