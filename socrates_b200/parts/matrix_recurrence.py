@@ -37,6 +37,9 @@ from .linear import Linear
 class MatrixRecurrence(Part):
     """What the two share: sizes, the kernel's scratch, the norm with its gate."""
     out_buffer = "branch"
+    # These mixers have been run with kernels launched strictly one after the other only (every model measured with
+    # them has routed experts, which ask for that): a model without such experts keeps to it.
+    serial_launches = True
 
     def _sizes(self, H: int, dk: int, dv: int, eps: float) -> None:
         self.H, self.dk, self.dv, self.eps = H, dk, dv, eps

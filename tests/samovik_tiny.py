@@ -84,6 +84,9 @@ TINY = {
     "F": ({"architecture": "Samovik", "vocab": 61, "width": 72, "norm": {"eps": 1e-5}, "token_side": {"dim": 8},
            "layers": [_layer("latent_attention", _lat(5, 16, 24, 32, 264, 0.3, 800.0), _moe(16, 1.0, 5, 2, (24, 1.0))),
                       _layer("latent_attention", _lat(6, 16, 8, 16, 40, 0.4, 60.0, (4.0, 30.0, 4.0, 1.0)), _moe(16, 1.0, 5, 2))]}, 8),
+    # no feed-forward anywhere, no cached rows
+    "G": ({"architecture": "Samovik", "vocab": 45, "width": 32, "norm": {"eps": 1e-5}, "token_side": {"dim": 8},
+           "layers": [_layer("wkv", _wkv(4, 16), None), _layer("lightning", _lin(2, 24, 16, [0.95, 0.8]), None)]}, 12),
 }
 
 

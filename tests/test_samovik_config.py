@@ -154,7 +154,9 @@ def test_plain_experts_and_clear_routing():
             plain.forward(cfg, w, ids.tolist())
         finally:
             plain.choose = original
-        assert min(gaps) > 0.03, (name, gaps)
+        assert min(gaps, default=1.0) > 0.03, (name, gaps)
+        if not gaps:
+            continue                                     # no routers in this one
         routed = [l["mlp"]["router"] for l in cfg["layers"] if l["mlp"]]
         assert len(seen) > sum(min(r["experts"], r["top"] + 1) for r in routed) - len(routed), name    # choices vary
     assert CODE == 6
