@@ -603,7 +603,8 @@ def run_compare(args):
             "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak",
             "vs_baseline": None, "dtype": "bf16",
             "data": "synthetic: random weights, token ids uniform over the vocabulary",
-            "config": {"model": f"{args.compare.capitalize()} and Qwen3 decoders at equal width and layer runs", "global_batch": B,
+            "config": {"model": f"{args.compare.capitalize()} and {'Loletar and ' if args.compare == 'samovik' else ''}Qwen3 decoders "
+                                f"at equal width and layer runs", "global_batch": B,
                        "seq_len": ctx, "prefill_tokens": T, "parallelism": "single GPU", "cuda_graph": True,
                        "l2": "inputs larger than L2 at widths 2k and 4k; a step's weights at 1k are not"},
             "clocks": sampler.summary(t_begin, t_end), "gpu_launches": launches, "impl": "ours", "compare": rows_out}
@@ -618,6 +619,8 @@ def model_tensors(model):
     def walk(obj, depth=0):
         import torch
         if isinstance(obj, torch.Tensor):
+            if obj._base is not None and obj._base.data_ptr() in seen:
+                return                                    # a slice of a tensor that is counted whole
             if obj.data_ptr() not in seen:
                 seen.add(obj.data_ptr())
                 out.append(obj)
@@ -656,7 +659,8 @@ def main():
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
     ap.add_argument("--compare", default=None, choices=("bofusun", "loletar", "samerax", "magedra", "samovik"),
-                    help="the Bofusun, the Loletar, the Samerax or the Magedra design at real layer widths beside Qwen3 at equal size "
+                    help="the Bofusun, the Loletar, the Samerax, the Magedra or the Samovik design at real layer widths beside Qwen3 at "
+                         "equal size "
                          "(prefill and decode); the default workload is not run")
     ap.add_argument("--only", default=None, help="with --compare: run only these of the pair, e.g. 'loletar' or 'qwen3'")
     ap.add_argument("--sizes", default=None, help="with --compare: widths to run, of 1k,2k,4k (default 1k,2k)")

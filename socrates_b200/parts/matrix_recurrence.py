@@ -117,6 +117,7 @@ class TokenShiftMixing(MatrixRecurrence):
         D = int(p["head_dim"])
         self._sizes(int(p["num_heads"]), D, D, float(p["norm_eps"]))
         self.rank_drawn = int(p.get("decay_rank", 64))        # of random weights; a checkpoint's tensors say theirs
+        self.rkvg: Optional[Linear] = None
         self.linears: Dict[str, Linear] = {}
         self.mu = self.w0 = self.u = None
 
@@ -135,7 +136,10 @@ class TokenShiftMixing(MatrixRecurrence):
     def bind(self, tensors: Mapping[str, torch.Tensor], dtype) -> None:
         n = self.name
         self.mu = torch.stack([tensors[f"{n}mu.{s}"] for s in self.MIXES]).contiguous()
-        self.linears = {s: Linear(tensors[n + s]) for s in ("r", "k", "v", "g", "w1", "w2")}
+        # r, k, v and g side by side: one product for a few tokens, four (of slices of the same tensor) for many
+        self.rkvg = Linear(torch.cat([tensors[n + s] for s in "rkvg"], dim=0))
+        self.linears = {s: Linear(self.rkvg.weight[i * self.Ck:(i + 1) * self.Ck]) for i, s in enumerate("rkvg")}
+        self.linears.update({s: Linear(tensors[n + s]) for s in ("w1", "w2")})
         if self.linears["w1"].out_features != self.linears["w2"].in_features:
             raise ValueError(f"{n}w1 has {self.linears['w1'].out_features} rows and {n}w2 "
                              f"{self.linears['w2'].in_features} columns; they are the decay's rank and must agree")
@@ -147,7 +151,7 @@ class TokenShiftMixing(MatrixRecurrence):
                                  "x": StateSpec((1, self.hidden), torch.float32)})
 
     def streamed_weights(self):
-        return [*(l.weight for l in self.linears.values()), self.o.weight]
+        return [self.rkvg.weight, self.linears["w1"].weight, self.linears["w2"].weight, self.o.weight]
 
     def forward(self, ctx, x: torch.Tensor, cache) -> Branch:
         N, d = x.shape
@@ -155,14 +159,23 @@ class TokenShiftMixing(MatrixRecurrence):
         mixed = ctx.buffers.take_flat("rec_mixes", len(self.MIXES) * N * d, ctx.dtype).view(len(self.MIXES), N, d)
         ops.token_shift_mix(mixed, x, self.mu, last, ctx.token_rows)
         ops.short_conv_tail(last, x, None, 2, ctx.seq_starts, ctx.seq_rows)       # the portion's last x stays
-        r, k, v, g = (self.linears[s](ctx, mixed[i], f"rec_{s}", out="model_or_partial") for i, s in enumerate("rkvg"))
+        C = self.Ck
+        stacked = mixed[:4].view(4 * N, d)
+        if 4 * N <= 64 and ctx.gemm_splits(4 * N, self.rkvg.weight, ctx.dtype) > 1:
+            # A few tokens: the product streams the weights whatever it multiplies, so all four blends go through all
+            # four matrices at once and every reader takes the block that is its own.
+            y = self.rkvg(ctx, stacked, "rec_rkvg", out="partial")                  # [S, 4 N, 4 C]
+            (r, r0), (k, k0), (v, v0), (g, g0) = ((y[:, i * N:(i + 1) * N], i * C) for i in range(4))
+        else:
+            r, k, v, g = (self.linears[s](ctx, mixed[i], f"rec_{s}", out="model_or_partial") for i, s in enumerate("rkvg"))
+            r0 = k0 = v0 = g0 = 0
         low = self.linears["w1"](ctx, mixed[4], "rec_w1", out="model_or_partial")
         act = ctx.buffers.take("rec_w1_act", N, (self.linears["w1"].out_features,), ctx.dtype)
         ops.bias_act(act, low, None, "tanh")
         raw_decay = self.linears["w2"](ctx, act, "rec_decay", out="float32")
-        raw = self._walk(ctx, N, (r, 0), (k, 0), (v, 0), cache.state("S"), raw_decay=(raw_decay, 0), decay_base=self.w0,
+        raw = self._walk(ctx, N, (r, r0), (k, k0), (v, v0), cache.state("S"), raw_decay=(raw_decay, 0), decay_base=self.w0,
                          bonus=self.u)
-        return self._finish(ctx, raw, (g, 0), self.H, "silu")
+        return self._finish(ctx, raw, (g, g0), self.H, "silu")
 
 
 register_part("mixer", "token_shift_mixing", TokenShiftMixing)
