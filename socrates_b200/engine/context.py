@@ -212,14 +212,18 @@ class StepContext:
                 ops.gemm_tcgen05(out, x, w, self.status, S, variant=ops.SHARES_VARIANT)
                 return
             ops.gemm_tcgen05(out if out.dim() == 3 and S > 1 else out.view(out.shape[-2], out.shape[-1]),
-                             x, w, self.status, S, epilogue=epilogue, prefetch=self._next_weights(w))
+                             x, w, self.status, S, epilogue=epilogue, prefetch=self._next_weights(w, S))
         else:
             if epilogue:
                 raise ValueError("the fused epilogue exists only in the tensor-core kernel")
             ops.gemm_simt(out, x, w, splits=S)
 
-    def _next_weights(self, w: torch.Tensor):
+    def _next_weights(self, w: torch.Tensor, splits: int):
         nxt = self.weight_successor.get(w.data_ptr())
         if nxt is None or self.l2_prefetch_bytes <= 0 or not nxt.is_contiguous():
             return None
-        return (nxt, self.l2_prefetch_bytes)
+        # A product of a few blocks (a narrow matrix) asks for little: the whole budget through sixteen blocks kept
+        # such a product on the GPU for 20 us instead of 5.
+        blocks = -(-w.shape[0] // 128) * splits
+        budget = self.l2_prefetch_bytes if blocks >= 64 else self.l2_prefetch_bytes * blocks // 256
+        return (nxt, budget)
