@@ -12,8 +12,8 @@ all layers, host-side lengths, and assign / release / move_row.  What is added h
   written (the reference reserves the worst case at admission,
   model/inference_paged.py:150-157).  It either takes every page it needs in every
   group or changes nothing.
-* **Windows give pages back.**  `commit(row, new_len)` frees the pages of a windowed
-  group that no later query can see.
+* **Windows and chunks give pages back.**  `commit(row, new_len)` frees the pages of a
+  windowed or chunked group that no later query can see.
 * **State slots.**  A mixer may ask for a fixed-size tensor per request; it lives at
   the request's row in `[max_rows, *shape]`, is zeroed on `assign`, and moves with
   `move_row`.
@@ -36,12 +36,33 @@ from .allocator import OutOfPages, PageAllocator, pages_for
 class PagedKVSpec:
     """Keys and values of `num_kv_heads` heads; keys have `head_dim` dims, values
     `v_head_dim` (None: the same); `window` keys are kept (None: all of them), and beside
-    the window the first `keep_first` keys of the sequence."""
+    the window the first `keep_first` keys of the sequence.  `chunk` (instead of a window): a query sees
+    the keys of its own chunk only, positions counted from the start of the sequence."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
+
+    def __post_init__(self):
+        if self.chunk is not None and (self.window is not None or self.chunk < 1):
+            raise ValueError(f"chunks of {self.chunk} keys beside a window of {self.window}")
+
+    @property
+    def bounded(self) -> bool:
+        """Whether keys fall out of sight as the sequence grows."""
+        return self.window is not None or self.chunk is not None
+
+    def most_keys(self) -> Optional[int]:
+        """The most keys at the end of a row that can be in sight (the newest one included); None: all of them."""
+        return self.chunk if self.chunk is not None else self.window
+
+    def first_visible(self, pos: int) -> int:
+        """The first position that a query at `pos` sees (beside the kept first keys)."""
+        if self.chunk is not None:
+            return pos - pos % self.chunk
+        return 0 if self.window is None else max(0, pos - self.window + 1)
 
     @property
     def value_dim(self) -> int:
@@ -96,9 +117,7 @@ class PageGroup:
 
     def first_needed_block(self, next_pos: int) -> int:
         """The lowest logical block that a query at `next_pos` or later can still see."""
-        if self.spec.window is None:
-            return 0
-        return max(0, next_pos - self.spec.window + 1) // self.page_size
+        return self.spec.first_visible(next_pos) // self.page_size
 
     def kept_blocks(self) -> int:
         """Logical blocks at the start of a row that a windowed group never gives back: those that
@@ -236,7 +255,7 @@ class CacheManager:
             raise ValueError("a row does not shrink")
         self.lengths[row] = new_len
         for g in self.groups:
-            if g.spec.window is None:
+            if not g.spec.bounded:
                 continue
             keep_from = g.first_needed_block(new_len)
             have = g.row_pages[row]

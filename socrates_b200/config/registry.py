@@ -12,6 +12,7 @@ from pathlib import Path
 from typing import Any, Dict, Mapping
 
 from .bofusun import BofusunConfig
+from .kusirax import KusiraxConfig
 from .loletar import LoletarConfig
 from .magedra import MagedraConfig
 from .qwen3 import ConfigError, Qwen3Config
@@ -65,3 +66,4 @@ register_architecture(LoletarConfig.architecture, LoletarConfig)
 register_architecture(SameraxConfig.architecture, SameraxConfig)
 register_architecture(MagedraConfig.architecture, MagedraConfig)
 register_architecture(SamovikConfig.architecture, SamovikConfig)
+register_architecture(KusiraxConfig.architecture, KusiraxConfig)

@@ -5,7 +5,8 @@
 //   s_ij = (q_i . k_j) * scale
 //   s_ij = cap * tanh(s_ij / cap)                  (cap > 0)
 //   s_ij += dist_bias[h][min(i - j, L - 1)]        (a table by distance, made on the host)
-//   keys j with 0 <= i - j < window                (window 0: all keys)
+//   s_ij -= slope_h * (i - j)                       (slopes optional)
+//   keys j with 0 <= i - j < window                (window 0: all keys), or those of i's own chunk of `chunk` positions
 //   o_i = softmax_j(s_ij) v_j * sigmoid(gate_i[h]) (gate optional; one per head, or one per head and value dim)
 //   with a sink: p_ij = exp(s_ij) / (exp(sink) + sum_j exp(s_ij)), one more term in the denominator that has no value
 //
@@ -15,6 +16,7 @@
 #include <math.h>
 
 #include "common.cuh"
+#include "score_map.cuh"
 #include "attention_reduce.cuh"
 
 using namespace sb;
@@ -47,6 +49,8 @@ struct BiasAttnArgs {
     int gate_per_dim;          // 0: gate column h; 1: gate column h * Dv + value dim
     int has_sink;              // the softmax denominator holds exp(sink) beside the keys' terms
     float sink;
+    const float* slopes;       // [Hq] or null: what a key loses per position of distance
+    int chunk;                 // > 0: only keys of the query's own chunk
 };
 
 // The sigmoid gate of output (token n, head h, value dim d); 1 without a gate.
@@ -71,7 +75,7 @@ __global__ void __launch_bounds__(THREADS) bias_attention_kernel(BiasAttnArgs a)
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int G = a.Hq / a.Hkv, Dk = a.Dk, Dv = a.Dv, BS = a.BS;
     const int row = a.token_rows[n], pos = a.positions[n];
-    const int lo_all = (a.window > 0 && pos + 1 > a.window) ? pos + 1 - a.window : 0;
+    const int lo_all = first_visible(pos, a.window, a.chunk);
     // this block's share of the visible keys lo_all..pos: equal counts, in order
     const int per = (pos + 1 - lo_all + a.NP - 1) / a.NP;
     const int lo = lo_all + (int)blockIdx.z * per;
@@ -135,6 +139,7 @@ __global__ void __launch_bounds__(THREADS) bias_attention_kernel(BiasAttnArgs a)
                     float s = dot[g] * a.scale;
                     if (a.cap > 0.f) s = a.cap * tanhf(s / a.cap);
                     if (a.dist_bias) s += a.dist_bias[(size_t)(h0 + g) * a.L + dist];
+                    if (a.slopes) s -= a.slopes[h0 + g] * (float)(pos - key);
                     w[g][tid] = s;
                 }
             }
@@ -254,7 +259,7 @@ __global__ void __launch_bounds__(THREADS, 4) bias_attention_tile_kernel(TileArg
     const int n_first = ta.seq_starts[r] + ti * QT;
     const int nq = min(QT, ta.seq_starts[r + 1] - n_first);                 // queries in this tile
     const int pos_first = ta.seq_first_pos[r] + ti * QT, pos_last = pos_first + nq - 1;
-    const int lo_tile = (a.window > 0 && pos_first + 1 > a.window) ? pos_first + 1 - a.window : 0;
+    const int lo_tile = first_visible(pos_first, a.window, a.chunk);
     const int* table = a.block_table + (size_t)ta.seq_rows[r] * a.table_width;
     const T* q = (const T*)a.q;
     const T* kp = (const T*)a.k_pool;
@@ -304,12 +309,13 @@ __global__ void __launch_bounds__(THREADS, 4) bias_attention_tile_kernel(TileArg
                 for (int row = 0; row < ROWS; ++row) {
                     const int qi = row / GP, g = row - qi * GP;
                     const int pos = pos_first + qi;
-                    const int lo = (a.window > 0 && pos + 1 > a.window) ? pos + 1 - a.window : 0;
+                    const int lo = first_visible(pos, a.window, a.chunk);
                     float sc = -INFINITY;
                     if (have && qi < nq && g < gn && key >= lo && key <= pos) {
                         sc = dot[row] * a.scale;
                         if (a.cap > 0.f) sc = a.cap * tanhf(sc / a.cap);
                         if (a.dist_bias) sc += a.dist_bias[(size_t)(h0 + g) * a.L + min(pos - key, a.L - 1)];
+                        if (a.slopes) sc -= a.slopes[h0 + g] * (float)(pos - key);
                     }
                     Ps[row * KEYS + tid] = sc;
                 }
@@ -377,14 +383,15 @@ extern "C" int sb_attention_bias(void* out, const void* q, const void* k_pool, c
                                  const float* dist_bias, int L, int N, int Hq, int Hkv, int Dk, int Dv,
                                  int page_size, int window, float scale, float cap, int num_partitions,
                                  float* part_o, float* part_ml, int dtype, int gate_per_dim, int has_sink,
-                                 float sink, cudaStream_t stream) {
+                                 float sink, const float* slopes, int chunk, cudaStream_t stream) {
     SB_REQUIRE(N >= 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0,
                "attention_bias: %d query heads are no multiple of %d KV heads", Hq, Hkv);
     SB_REQUIRE(Dk >= 1 && Dk <= DMAX && Dv >= 1 && Dv <= 4 * THREADS,
                "attention_bias: head sizes %d (keys, at most %d) and %d (values, at most %d)", Dk, DMAX, Dv, 4 * THREADS);
     SB_REQUIRE(page_size > 0 && table_width > 0, "attention_bias: bad page_size %d or table width %d", page_size,
                table_width);
-    SB_REQUIRE(window >= 0, "attention_bias: window %d is negative", window);
+    SB_REQUIRE(window >= 0 && chunk >= 0 && !(window > 0 && chunk > 0),
+               "attention_bias: a window of %d and chunks of %d", window, chunk);
     SB_REQUIRE(dist_bias == nullptr || L >= 1, "attention_bias: a bias table needs a length");
     SB_REQUIRE(N <= 65535, "attention_bias: %d tokens exceed one launch", N);
     SB_REQUIRE(num_partitions >= 1 && num_partitions <= 64 &&
@@ -397,7 +404,7 @@ extern "C" int sb_attention_bias(void* out, const void* q, const void* k_pool, c
     a.gate_stride = gate_stride; a.dist_bias = dist_bias; a.L = L > 0 ? L : 1; a.Hq = Hq; a.Hkv = Hkv; a.Dk = Dk;
     a.Dv = Dv; a.BS = page_size; a.window = window; a.scale = scale; a.cap = cap;
     a.NP = num_partitions; a.part_o = part_o; a.part_ml = part_ml;
-    a.gate_per_dim = gate_per_dim; a.has_sink = has_sink; a.sink = sink;
+    a.gate_per_dim = gate_per_dim; a.has_sink = has_sink; a.sink = sink; a.slopes = slopes; a.chunk = chunk;
     dim3 grid(Hkv, N, num_partitions), rgrid(Hq, N);
     if (dtype == SB_F32) {
         if (Dv > 2 * THREADS) sb::launch(bias_attention_kernel<float, 4>, grid, dim3(THREADS), 0, stream, a);
@@ -429,7 +436,9 @@ extern "C" int sb_attention_bias_tile(void* out, const void* q, const void* k_po
                                       const int* seq_rows, const int* seq_first_pos, int R, const void* gate,
                                       long long gate_stride, const float* dist_bias, int L, int N, int Hq, int Hkv,
                                       int Dk, int Dv, int page_size, int window, float scale, float cap, int dtype,
-                                      int gate_per_dim, int has_sink, float sink, cudaStream_t stream) {
+                                      int gate_per_dim, int has_sink, float sink, const float* slopes, int chunk,
+                                      cudaStream_t stream) {
+    SB_REQUIRE(chunk >= 0 && !(window > 0 && chunk > 0), "attention_bias_tile: a window of %d and chunks of %d", window, chunk);
     SB_REQUIRE(sb_attention_bias_tile_supports(Hq, Hkv, Dk, Dv, dtype),
                "attention_bias_tile: heads %d/%d of %d (keys) and %d (values) are not served", Hq, Hkv, Dk, Dv);
     SB_REQUIRE((reinterpret_cast<uintptr_t>(k_pool) & 15) == 0, "attention_bias_tile: the key pool must be 16-byte aligned");
@@ -444,7 +453,7 @@ extern "C" int sb_attention_bias_tile(void* out, const void* q, const void* k_po
     a.gate_stride = gate_stride; a.dist_bias = dist_bias; a.L = L > 0 ? L : 1; a.Hq = Hq; a.Hkv = Hkv; a.Dk = Dk;
     a.Dv = Dv; a.BS = page_size; a.window = window; a.scale = scale; a.cap = cap; a.NP = 1; a.part_o = nullptr;
     a.part_ml = nullptr;
-    a.gate_per_dim = gate_per_dim; a.has_sink = has_sink; a.sink = sink;
+    a.gate_per_dim = gate_per_dim; a.has_sink = has_sink; a.sink = sink; a.slopes = slopes; a.chunk = chunk;
     ta.seq_starts = seq_starts; ta.seq_rows = seq_rows; ta.seq_first_pos = seq_first_pos; ta.R = R;
     ta.GP = G >= 4 ? 4 : (G >= 2 ? 2 : 1);
     ta.QT = ROWS / ta.GP;

@@ -27,6 +27,7 @@
 #include "attention_reduce.cuh"
 
 #include "attention_mma.cuh"
+#include "score_map.cuh"
 
 extern "C" int sb_attention_decode_mma_kernels(int num_partitions);
 
@@ -150,13 +151,23 @@ attn_prefill_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, const bf
 // CLUSTER: the NP blocks of a (token, KV head) are one thread-block cluster and merge their
 // partial results through distributed shared memory: no scratch in global memory, no reduce
 // kernel.  Every block of the cluster reaches both cluster barriers (an empty partition too).
-template <int D, int NW, int S, bool CLUSTER = false, int NBQ = 1>
+// MAPPED: scores are capped and / or lose a slope times the distance (score_map.cuh); `scale_log2` is the plain
+// scale then.
+template <int NBQ> struct ColumnMap {
+    sb::RowScores row[2 * NBQ];
+    int pos;
+    __device__ __forceinline__ float operator()(float s, int key, int nb, int e) const {
+        return row[2 * nb + e](s, (float)(key - pos));
+    }
+};
+
+template <int D, int NW, int S, bool CLUSTER = false, int NBQ = 1, bool MAPPED = false>
 __global__ void __launch_bounds__(32 * NW)
 attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                    const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                    const int* __restrict__ block_table, int table_width, const int* __restrict__ token_rows,
                    const int* __restrict__ positions, int Hq, int Hkv, int BS, int window, float scale_log2,
-                   int NP) {
+                   int NP, sb::ScoreMap score_map) {
     sb::pdl_launch_dependents();     // the next kernel may begin its prologue
     // What is read before pdl_wait() below was complete before the preceding kernel began:
     // the block table, rows and positions (copied from the host at the start of the step)
@@ -179,7 +190,7 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     const int pos = positions[n];
     const int* table = block_table + (size_t)token_rows[n] * table_width;
     const int hi = pos + 1;
-    const int lo = (window > 0 && hi > window) ? hi - window : 0;
+    const int lo = sb::first_visible(pos, window, score_map.chunk);
     const int first_pg = lo / BS, last_pg = (hi - 1) / BS;
     const int ppp = (last_pg - first_pg + 1 + NP - 1) / NP;
     const int pg_begin = first_pg + part * ppp;
@@ -187,6 +198,14 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     const int k_begin = max(lo, pg_begin * BS);
     const int k_end = min(hi, pg_end * BS);
     const int h0 = kh * G;
+    const float per_unit = MAPPED ? 1.0f : scale_log2;      // from scores to exponents of 2
+    ColumnMap<NBQ> col_map;
+    if constexpr (MAPPED) {                                 // the thread's columns are query heads 2 (lane % 4), + 1
+        col_map.pos = pos;
+#pragma unroll
+        for (int c = 0; c < 2 * NBQ; ++c)
+            col_map.row[c].set(score_map, scale_log2, h0 + min(G - 1, 8 * (c >> 1) + 2 * (lane & 3) + (c & 1)));
+    }
 
     const bool empty = k_begin >= k_end;                    // an empty partition (only when NP > 1)
     if (empty && CLUSTER) {
@@ -258,8 +277,12 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
                                                 v_pool, stab, pg_begin, bs_log2, Hkv, kh, (tile_begin + nxt) * KTD,
                                                 k_begin, k_end);
         };
-        warp_tile_decode<D, NBQ>(st, qf, kbuf + buf * KTD * D, vbuf + buf * KTD * D, warp * 16, ts, pos, k_begin,
-                                 k_end, scale_log2, masked, between);
+        if constexpr (MAPPED)
+            warp_tile_decode<D, NBQ>(st, qf, kbuf + buf * KTD * D, vbuf + buf * KTD * D, warp * 16, ts, pos, k_begin,
+                                     k_end, per_unit, masked, between, col_map);
+        else
+            warp_tile_decode<D, NBQ>(st, qf, kbuf + buf * KTD * D, vbuf + buf * KTD * D, warp * 16, ts, pos, k_begin,
+                                     k_end, per_unit, masked, between);
         cp_async_commit();
     }
     cp_async_wait<0>();
@@ -303,7 +326,7 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
         float L = 0.f, o = 0.f;
 #pragma unroll
         for (int w = 0; w < NW; ++w) {
-            const float f = wl[w] > 0.f ? ex2_approx((wm[w] - M) * scale_log2) : 0.f;
+            const float f = wl[w] > 0.f ? ex2_approx((wm[w] - M) * per_unit) : 0.f;
             L += f * wl[w];
             o += wl[w] > 0.f ? f * wv[w] : 0.f;
         }
@@ -313,14 +336,14 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
         } else if (CLUSTER) {
             wo[(size_t)NW * 16 * D + idx] = o;              // behind the warps' rows: [G][D] of this partition
             if (d == 0) {
-                c_ml[row][0] = M * scale_log2 / LOG2E;      // natural exponents, as in the reduce kernel
+                c_ml[row][0] = M * per_unit / LOG2E;      // natural exponents, as in the reduce kernel
                 c_ml[row][1] = L;
             }
         } else {
             part_o[(((size_t)n * Hq + h) * NP + part) * D + d] = o;
             if (d == 0) {
                 float* ml = part_ml + (((size_t)n * Hq + h) * NP + part) * 2;
-                ml[0] = M * scale_log2 / LOG2E;             // natural exponents, as the reduce kernel expects
+                ml[0] = M * per_unit / LOG2E;             // natural exponents, as the reduce kernel expects
                 ml[1] = L;
             }
         }
@@ -406,33 +429,34 @@ inline bool cluster_merge_enabled() {
     return on;
 }
 
-template <int D, int NW, int S, int NBQ>
+template <int D, int NW, int S, int NBQ, bool MAPPED>
 int launch_decode_v(void* out, float* part_o, float* part_ml, const void* q, const void* k_pool, const void* v_pool,
                     const int* block_table, int table_width, const int* token_rows, const int* positions, int N,
-                    int Hq, int Hkv, int BS, int window, float scale, int NP, cudaStream_t stream) {
+                    int Hq, int Hkv, int BS, int window, float scale, int NP, const sb::ScoreMap& map, cudaStream_t stream) {
     constexpr int smem = decode_smem<D, NW, S>();
     const bool cluster = NP >= 2 && sb_attention_decode_mma_kernels(NP) == 1;
     static sb::OncePerDevice once_per_device;
     bool& configured = once_per_device.flag();
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D, NW, S, false, NBQ>,
+        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<D, NW, S, false, NBQ, MAPPED>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, smem + kMaxTableWidth * 4);
         if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(attn_decode_kernel<D, NW, S, true, NBQ>,
+            e = cudaFuncSetAttribute(attn_decode_kernel<D, NW, S, true, NBQ, MAPPED>,
                                      cudaFuncAttributeMaxDynamicSharedMemorySize, smem + kMaxTableWidth * 4);
         if (e != cudaSuccess) { sb_set_error("attention_mma: %s", cudaGetErrorString(e)); return (int)e; }
         configured = true;
     }
     dim3 grid(Hkv, N, NP);
     if (cluster) {
-        sb::launch_cluster(attn_decode_kernel<D, NW, S, true, NBQ>, dim3(grid), dim3(32 * NW), smem + table_width * 4, stream,
+        sb::launch_cluster(attn_decode_kernel<D, NW, S, true, NBQ, MAPPED>, dim3(grid), dim3(32 * NW), smem + table_width * 4, stream,
             dim3(1, 1, NP), (bf16*)out, part_o, part_ml, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool,
-            block_table, table_width, token_rows, positions, Hq, Hkv, BS, window, scale * LOG2E, NP);
+            block_table, table_width, token_rows, positions, Hq, Hkv, BS, window,
+            MAPPED ? scale : scale * LOG2E, NP, map);
         return 0;
     }
-    sb::launch(attn_decode_kernel<D, NW, S, false, NBQ>, dim3(grid), dim3(32 * NW), smem + table_width * 4, stream, 
+    sb::launch(attn_decode_kernel<D, NW, S, false, NBQ, MAPPED>, dim3(grid), dim3(32 * NW), smem + table_width * 4, stream, 
         (bf16*)out, part_o, part_ml, (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table,
-        table_width, token_rows, positions, Hq, Hkv, BS, window, scale * LOG2E, NP);
+        table_width, token_rows, positions, Hq, Hkv, BS, window, MAPPED ? scale : scale * LOG2E, NP, map);
     if (NP > 1) {
         dim3 rgrid(Hq, N);
         sb::launch(attn_reduce_kernel<bf16>, dim3(rgrid), dim3(128), 0, stream, (bf16*)out, part_o, part_ml, Hq, D, NP);
@@ -450,14 +474,18 @@ constexpr int kVariantStages[kDecodeVariants] = {3, 2};
 template <int D>
 int launch_decode(void* out, float* part_o, float* part_ml, const void* q, const void* k_pool, const void* v_pool,
                   const int* block_table, int table_width, const int* token_rows, const int* positions, int N,
-                  int Hq, int Hkv, int BS, int window, float scale, int NP, cudaStream_t stream, int variant = 0) {
-#define SB_DEC(NW, S, NBQ) launch_decode_v<D, NW, S, NBQ>(out, part_o, part_ml, q, k_pool, v_pool, block_table, \
+                  int Hq, int Hkv, int BS, int window, float scale, int NP, cudaStream_t stream, int variant = 0,
+                  const sb::ScoreMap& map = sb::ScoreMap{0.f, nullptr, 0}) {
+#define SB_DEC_(NW, S, NBQ, MAPPED) launch_decode_v<D, NW, S, NBQ, MAPPED>(out, part_o, part_ml, q, k_pool, v_pool, block_table, \
                                                           table_width, token_rows, positions, N, Hq, Hkv, BS, window, \
-                                                          scale, NP, stream)
+                                                          scale, NP, map, stream)
+#define SB_DEC(NW, S, NBQ) SB_DEC_(NW, S, NBQ, false)
+    if (map.maps_scores()) return Hq / Hkv <= 8 ? SB_DEC_(4, 3, 1, true) : SB_DEC_(4, 3, 2, true);
     // query heads of a KV head: one block of 8 columns, or two
     if (Hq / Hkv <= 8) return variant == 1 ? SB_DEC(4, 2, 1) : SB_DEC(4, 3, 1);
     return variant == 1 ? SB_DEC(4, 2, 2) : SB_DEC(4, 3, 2);
 #undef SB_DEC
+#undef SB_DEC_
 }
 
 }  // namespace
@@ -511,7 +539,8 @@ extern "C" int sb_attention_decode_mma_blocks_per_sm(int D, int variant) {
 }
 
 // Steps in which every request brings one token.  Scratch as for sb_attention_simt.
-// `variant` selects (warps, stages) of the kernel; 0 is the default.
+// `variant` selects (warps, stages) of the kernel; 0 is the default (and the only one with mapped scores).
+// `cap`, `slopes` [Hq] and `chunk`: see score_map.cuh (0 / null: none).
 // The block table, rows, positions, and keys and values below each token's position must be
 // complete before the kernel that precedes this one on the stream started; the query and
 // the newest key and value may come from that kernel.
@@ -519,7 +548,11 @@ extern "C" int sb_attention_decode_mma(void* out, float* part_o, float* part_ml,
                                        const void* k_pool, const void* v_pool, const int* block_table,
                                        int table_width, const int* token_rows, const int* positions, int N,
                                        int Hq, int Hkv, int D, int page_size, int window, float scale,
-                                       int num_partitions, int variant, cudaStream_t stream) {
+                                       int num_partitions, int variant, float cap, const float* slopes, int chunk,
+                                       cudaStream_t stream) {
+    SB_REQUIRE(cap >= 0.f && chunk >= 0 && !(chunk > 0 && window > 0),
+               "attention_mma: a cap of %f, chunks of %d beside a window of %d", (double)cap, chunk, window);
+    const sb::ScoreMap map{cap, slopes, chunk};
     SB_REQUIRE(sb_attention_mma_supports(Hq, Hkv, D, page_size, 1),
                "attention_mma (decode): Hq=%d Hkv=%d head_dim=%d is not supported", Hq, Hkv, D);
     SB_REQUIRE(N > 0 && N <= 65535 && window >= 0 && table_width > 0, "attention_mma: bad sizes N=%d", N);
@@ -530,10 +563,10 @@ extern "C" int sb_attention_decode_mma(void* out, float* part_o, float* part_ml,
                "attention_mma: split over %d partitions needs scratch buffers", num_partitions);
     int rc;
     switch (D) {
-        case 16: rc = launch_decode<16>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant); break;
-        case 32: rc = launch_decode<32>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant); break;
-        case 64: rc = launch_decode<64>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant); break;
-        default: rc = launch_decode<128>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant); break;
+        case 16: rc = launch_decode<16>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant, map); break;
+        case 32: rc = launch_decode<32>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant, map); break;
+        case 64: rc = launch_decode<64>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant, map); break;
+        default: rc = launch_decode<128>(out, part_o, part_ml, q, k_pool, v_pool, block_table, table_width, token_rows, positions, N, Hq, Hkv, page_size, window, scale, num_partitions, stream, variant, map); break;
     }
     if (rc != 0) return rc;
     SB_LAUNCH_CHECK();

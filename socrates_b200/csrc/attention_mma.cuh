@@ -280,11 +280,18 @@ template <int D, int NBQ> struct ColState {
 // One warp: its 16 keys (kb .. kb+15 of the tile at tile_start) against the token's query heads.
 //   qf: the query fragments as loaded for an A operand (rows 0-7 and 8-15, two 8-dim chunks).
 //   Keys outside [klo, khi) or beyond qpos are masked when `masked`.
+//   map(score, key position, column block, which of the thread's two columns): what happens to a raw score first
+//   (`scale_log2` = 1 then: mapped scores are in units of log2); NoMap leaves it alone.
 //   between(p), p = 0..3: called between the phases (the caller issues a later tile's copies there).
-template <int D, int NBQ, typename Between>
+struct NoMap {
+    __device__ __forceinline__ float operator()(float s, int, int, int) const { return s; }
+};
+
+template <int D, int NBQ, typename Between, typename Map = NoMap>
 __device__ __forceinline__ void warp_tile_decode(ColState<D, NBQ>& st, const uint32_t (&qf)[D / 16][4],
                                                  const bf16* ks, const bf16* vs, int kb, int tile_start, int qpos,
-                                                 int klo, int khi, float scale_log2, bool masked, Between between) {
+                                                 int klo, int khi, float scale_log2, bool masked, Between between,
+                                                 const Map& map = Map{}) {
     const int lane = threadIdx.x & 31;
     const int j = lane >> 3;
     // ---- S^T = K Q^T.  The D/16 products of a column block would be one chain through their
@@ -312,7 +319,7 @@ __device__ __forceinline__ void warp_tile_decode(ColState<D, NBQ>& st, const uin
             float v = sp[0][nb][e];
 #pragma unroll
             for (int c = 1; c < CH; ++c) v += sp[c][nb][e];
-            s[nb][e] = v;
+            s[nb][e] = map(v, tile_start + kb + (lane >> 2) + 8 * (e >> 1), nb, e & 1);
         }
     // ---- mask: the thread's keys are rows lane/4 and lane/4 + 8
     if (masked) {

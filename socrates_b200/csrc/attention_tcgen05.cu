@@ -37,6 +37,7 @@
 #include <stdint.h>
 
 #include "common.cuh"
+#include "score_map.cuh"
 #include "tma_maps.cuh"
 
 using namespace sb;
@@ -184,7 +185,9 @@ __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
 // that issues the P.V products
 constexpr int THREADS = ROWS + 96;
 
-template <int D>
+// MAPPED: scores are capped and / or lose a slope times the distance (see score_map.cuh); `scale_log2` is the
+// plain scale then, and a row's scores are turned into units of log2 as they are read.
+template <int D, bool MAPPED>
 __global__ void __launch_bounds__(THREADS)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
                             bf16* __restrict__ out, const bf16* __restrict__ q,
@@ -193,7 +196,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
                             const int* __restrict__ seq_first_pos, int R, int Hq, int Hkv, int BS, int window,
                             float scale_log2, int* __restrict__ status, const bf16* __restrict__ gate,
                             long long gate_stride, int gate_per_dim, int has_sink, float sink_raw, int keep_first,
-                            float* __restrict__ out_f32) {
+                            float* __restrict__ out_f32, ScoreMap map) {
     constexpr int PANELS = D / 64;                         // 64-dim panels of 128-byte rows
     constexpr int PANEL_Q = ROWS * 128;                    // bytes of one Q panel
     constexpr int PANEL_KV = KTILE * 128;                  // bytes of one K or V panel
@@ -263,7 +266,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
     if (active) {
         first_pos = seq_first_pos[r] + tile * TQ;
         hi = first_pos + n_tok;
-        lo = (window > 0 && first_pos + 1 > window) ? first_pos + 1 - window : 0;
+        lo = first_visible(first_pos, window, map.chunk);
         tile_begin = lo / KTILE;
         keep_tiles = min((kf + KTILE - 1) / KTILE, tile_begin);
         n_tiles = (hi + KTILE - 1) / KTILE - tile_begin + keep_tiles;
@@ -293,7 +296,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
     const uint32_t tmem = tmem_slot;
     // rows of this block see every key of a tile when it ends at or before the first query's
     // position and starts at or after the last query's window start
-    const int last_qlo = (window > 0 && hi > window) ? hi - window : 0;
+    const int last_qlo = active ? first_visible(hi - 1, window, map.chunk) : 0;
 
     if (copier) {
         // =============================================================== the copy-issuing warp
@@ -400,7 +403,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
         float m_ref = has_sink ? sink_raw : -INFINITY, l_run = has_sink ? 1.f : 0.f;
         const int tok = tid / G, g = tid - tok * G;
         const int qpos = tok < n_tok ? first_pos + tok : -1;   // rows past the tile see no key
-        const int qlo = (window > 0 && qpos + 1 > window) ? qpos + 1 - window : 0;
+        const int qlo = qpos >= 0 ? first_visible(qpos, window, map.chunk) : 0;
+        RowScores row_scores;
+        if constexpr (MAPPED) row_scores.set(map, scale_log2, kh * G + g);
+        const float per_unit = MAPPED ? 1.0f : scale_log2;     // from the scores below to exponents of 2
         const uint32_t lane_base = tmem + (static_cast<uint32_t>(warp * 32) << 16);
         bool ok = true;
         for (int i = 0; i < n_tiles; ++i) {
@@ -424,6 +430,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
 #pragma unroll
                 for (int j = 0; j < 32; ++j) s[32 + j] = __uint_as_float(raw[j]);
             }
+            if constexpr (MAPPED) {
+                const float ahead = (float)(tile_start - qpos);
+#pragma unroll
+                for (int j = 0; j < 64; ++j) s[j] = row_scores(s[j], ahead + (float)j);
+            }
             // position masks only where some row of the block cannot see some key of the tile;
             // rows past the tile (qpos = -1) are masked by the same test
             const bool masked = i < keep_tiles ? (tile_start + KTILE > kf || n_tok < TQ)
@@ -445,11 +456,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
             }
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
             // lazy rescale: move the reference maximum only when the row maximum outgrew it
-            const bool grow = mx > -INFINITY && (m_ref == -INFINITY || (mx - m_ref) * scale_log2 > RESCALE_LOG2);
+            const bool grow = mx > -INFINITY && (m_ref == -INFINITY || (mx - m_ref) * per_unit > RESCALE_LOG2);
             if (__any_sync(0xffffffffu, grow)) {
                 float alpha = 1.0f;
                 if (grow) {
-                    alpha = m_ref == -INFINITY ? 0.f : exp2f((m_ref - mx) * scale_log2);
+                    alpha = m_ref == -INFINITY ? 0.f : exp2f((m_ref - mx) * per_unit);
                     m_ref = mx;
                     l_run *= alpha;
                 }
@@ -476,15 +487,15 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
                 }
             }
             // p = 2^((s - m) * scale) as one multiply-add and one ex2; masked scores are -inf -> 0
-            const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref * scale_log2;
+            const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref * per_unit;
             float l4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int c = 0; c < KTILE; c += 32) {
                 uint32_t ph[16], pl[16];
 #pragma unroll
                 for (int j = 0; j < 16; ++j) {
-                    const float p0 = ex2_approx(fmaf(s[c + 2 * j], scale_log2, neg_m));
-                    const float p1 = ex2_approx(fmaf(s[c + 2 * j + 1], scale_log2, neg_m));
+                    const float p0 = ex2_approx(fmaf(s[c + 2 * j], per_unit, neg_m));
+                    const float p1 = ex2_approx(fmaf(s[c + 2 * j + 1], per_unit, neg_m));
                     l4[j & 3] += p0 + p1;
                     const uint32_t h = pack_bf16(p0, p1);
                     ph[j] = h;
@@ -610,12 +621,13 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
     }
 }
 
-template <int D>
+template <int D, bool MAPPED>
 int launch(const CUtensorMap& mk, const CUtensorMap& mv, void* out, const void* q, const int* block_table,
            int table_width, const int* seq_starts, const int* seq_rows, const int* seq_first_pos, int R, int N,
            int Hq, int Hkv, int BS, int window, float scale, int* status, const void* gate, long long gate_stride,
-           int gate_per_dim, int has_sink, float sink, int keep_first, float* out_f32, cudaStream_t stream) {
-    auto kernel = attn_prefill_tcgen05_kernel<D>;
+           int gate_per_dim, int has_sink, float sink, int keep_first, float* out_f32, const ScoreMap& map,
+           cudaStream_t stream) {
+    auto kernel = attn_prefill_tcgen05_kernel<D, MAPPED>;
     static sb::OncePerDevice once_per_device;
     bool& configured = once_per_device.flag();
     if (!configured) {
@@ -628,8 +640,8 @@ int launch(const CUtensorMap& mk, const CUtensorMap& mv, void* out, const void* 
     dim3 grid((N / TQ + R) * Hkv);                           // an upper bound of the number of tiles, times heads
     sb::launch(kernel, grid, dim3(THREADS), smem_bytes<D>() + table_width * 4, stream, mk, mv, (bf16*)out,
                (const bf16*)q, block_table, table_width, seq_starts, seq_rows, seq_first_pos, R, Hq, Hkv, BS, window,
-               scale * LOG2E, status, (const bf16*)gate, gate_stride, gate_per_dim, has_sink,
-               has_sink ? sink / scale : 0.f, keep_first, out_f32);
+               MAPPED ? scale : scale * LOG2E, status, (const bf16*)gate, gate_stride, gate_per_dim, has_sink,
+               has_sink ? (MAPPED ? sink * LOG2E : sink / scale) : 0.f, keep_first, out_f32, map);
     return 0;
 }
 
@@ -648,14 +660,17 @@ extern "C" int sb_attention_tcgen05_supports(int Hq, int Hkv, int D, int page_si
 // (`gate` [N, gate_stride] bfloat16, one column per head, or per head and dim) and a sink (a score
 // whose exponential joins the denominator without a value); `keep_first`: a window also sees the first
 // so many keys of its row; `out_f32` (float32 [N, Hq*D], or null): the rows are written there unrounded
-// and ungated instead of to `out`.
+// and ungated instead of to `out`; `cap`, `slopes` [Hq] and `chunk` as in score_map.cuh (0 / null: none).
 extern "C" int sb_attention_prefill_tcgen05(void* out, const void* q, const void* k_pool, const void* v_pool,
                                             int num_pages, const int* block_table, int table_width,
                                             const int* seq_starts, const int* seq_rows,
                                             const int* seq_first_pos, int R, int N, int Hq, int Hkv, int D,
                                             int page_size, int window, float scale, int* status,
                                             const void* gate, long long gate_stride, int gate_per_dim, int has_sink,
-                                            float sink, int keep_first, float* out_f32, cudaStream_t stream) {
+                                            float sink, int keep_first, float* out_f32, float cap, const float* slopes,
+                                            int chunk, cudaStream_t stream) {
+    SB_REQUIRE(cap >= 0.f && chunk >= 0 && !(chunk > 0 && window > 0),
+               "attention_tcgen05: a cap of %f, chunks of %d beside a window of %d", (double)cap, chunk, window);
     SB_REQUIRE(keep_first >= 0, "attention_tcgen05: %d kept keys", keep_first);
     SB_REQUIRE(!has_sink || scale > 0.f, "attention_tcgen05: a sink needs a positive scale");
     if (gate != nullptr && gate_per_dim && (reinterpret_cast<uintptr_t>(gate) & 15) == 0 && gate_stride % 8 == 0)
@@ -672,13 +687,15 @@ extern "C" int sb_attention_prefill_tcgen05(void* out, const void* q, const void
         sb_set_error("attention_tcgen05: cuTensorMapEncodeTiled failed");
         return SB_ERR_ARG;
     }
+    const ScoreMap map{cap, slopes, chunk};
+#define SB_TILE(D_, MAPPED_) \
+    launch<D_, MAPPED_>(mk, mv, out, q, block_table, table_width, seq_starts, seq_rows, seq_first_pos, R, N, Hq, Hkv, \
+                        page_size, window, scale, status, gate, gate_stride, gate_per_dim, has_sink, sink, keep_first, \
+                        out_f32, map, stream)
     int rc;
-    if (D == 64)
-        rc = launch<64>(mk, mv, out, q, block_table, table_width, seq_starts, seq_rows, seq_first_pos, R, N, Hq, Hkv,
-                        page_size, window, scale, status, gate, gate_stride, gate_per_dim, has_sink, sink, keep_first, out_f32, stream);
-    else
-        rc = launch<128>(mk, mv, out, q, block_table, table_width, seq_starts, seq_rows, seq_first_pos, R, N, Hq,
-                         Hkv, page_size, window, scale, status, gate, gate_stride, gate_per_dim, has_sink, sink, keep_first, out_f32, stream);
+    if (map.maps_scores()) rc = D == 64 ? SB_TILE(64, true) : SB_TILE(128, true);
+    else rc = D == 64 ? SB_TILE(64, false) : SB_TILE(128, false);
+#undef SB_TILE
     if (rc != 0) return rc;
     SB_LAUNCH_CHECK();
 }

@@ -259,6 +259,24 @@ extern "C" int sb_add_rmsnorm(float* residual, const float* delta, int S, long l
 // first R dims.  `magnitude` multiplies every cosine and sine (an encoding that also scales the
 // rotated dims); dims that do not rotate are not scaled.  With `spread` the queries are written one
 // row per (head, map), [N, Hq * maps, D]: the map's dims where they are and zeros elsewhere.
+// With `unit` the norm of q and k has no gain.  Values that several layers share: the layer that makes them
+// (values 1) leaves its own in `v_first` (float32 [N, Hkv * Dv]) beside its pages; a layer that blends (values 2)
+// writes (1 - blend) * own + blend * v_first to its pages.
+struct QkExtra {
+    const float* bias;
+    int unit;
+    int values;
+    float blend;
+    float* v_first;
+
+    __host__ __device__ bool any() const { return bias != nullptr || unit || values != 0; }
+    // what reaches the pages for an own value `v` at index `at` of v_first
+    __device__ __forceinline__ float value(float v, size_t at) const {
+        if (values == 1) v_first[at] = v;
+        return values == 2 ? fmaf(blend, v_first[at], (1.0f - blend) * v) : v;
+    }
+};
+
 template <typename T>
 __global__ void __launch_bounds__(128, 6) qk_norm_rope_kvwrite_kernel(
     const T* __restrict__ qkv, const float* __restrict__ parts, int S, size_t part_stride,
@@ -267,7 +285,8 @@ __global__ void __launch_bounds__(128, 6) qk_norm_rope_kvwrite_kernel(
     const float* __restrict__ inv_freq, int R, const int* __restrict__ positions,
     const int* __restrict__ token_rows, const int* __restrict__ block_table, int table_width,
     int BS, float eps, int Hq, int Hkv, int D, int write_kv, int Dv, int row_width, int neighbours,
-    const float* __restrict__ bias, int sub, float magnitude, int spread, int hpb) {
+    QkExtra extra, int sub, float magnitude, int spread, int hpb) {
+    const float* __restrict__ bias = extra.bias;
     sb::pdl_launch_dependents();     // the next kernel may begin its prologue
     sb::pdl_wait();                  // everything before this kernel is complete and visible
     __shared__ float buf[4][256];
@@ -372,6 +391,10 @@ __global__ void __launch_bounds__(128, 6) qk_norm_rope_kvwrite_kernel(
             ss = warp_sum(ss);
             const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
             for (int i = lane; i < D; i += 32) y[i] = y[i] * rinv * gain[i];
+        } else if (extra.unit && !is_v) {
+            ss = warp_sum(ss);
+            const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
+            for (int i = lane; i < D; i += 32) y[i] *= rinv;
         }
         __syncwarp();
 
@@ -387,7 +410,8 @@ __global__ void __launch_bounds__(128, 6) qk_norm_rope_kvwrite_kernel(
         for (int u = 0; u < 8; ++u) {
             const int i = lane + 32 * u;
             if (i >= Dh) break;
-            const float o = is_v ? y[i] : y[i] * rc[u] + y[rmate[u]] * rs[u];
+            const float o = is_v ? extra.value(y[i], ((size_t)n * Hkv + (head - Hq - Hkv)) * Dv + i)
+                                 : y[i] * rc[u] + y[rmate[u]] * rs[u];
             if (is_q && spread && maps == 2) {
                 // a row per map: the map's dims in their place, zeros where the other map's dims are
                 dst[i] = from_float<T>(rmap[u] == 0 ? o : 0.f);
@@ -410,14 +434,16 @@ template <typename T, int VPL> struct alignas(sizeof(T) * VPL) Pack { T v[VPL]; 
 // finds its rotation partner (dim +- D/2) in lane l ^ 16.  A block serves `heads_per_block`
 // heads of one token; its first D/2 threads compute the token's cosines and sines once
 // into shared memory, so the trigonometry is not repeated for every head.
-template <typename T, int VPL>
+// EXTRA: what `QkExtra` holds, and rotations of the first R < D dims (R a multiple of 2 * VPL: a lane's
+// dims rotate together or not at all, and the partners are R / 2 / VPL lanes apart).
+template <typename T, int VPL, bool EXTRA>
 __global__ void qk_norm_rope_kvwrite_fast_kernel(
     const T* __restrict__ qkv, const float* __restrict__ parts, int S, size_t part_stride,
     T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool,
     const float* __restrict__ q_gain, const float* __restrict__ k_gain,
     const float* __restrict__ inv_freq, int R, const int* __restrict__ positions,
     const int* __restrict__ token_rows, const int* __restrict__ block_table, int table_width,
-    int BS, float eps, int Hq, int Hkv, int write_kv, int heads_per_block) {
+    int BS, float eps, int Hq, int Hkv, int write_kv, int heads_per_block, QkExtra extra) {
     sb::pdl_launch_dependents();     // the next kernel may begin its prologue
     constexpr int D = 32 * VPL;
     __shared__ float cs[D / 2], sn[D / 2];
@@ -425,8 +451,8 @@ __global__ void qk_norm_rope_kvwrite_fast_kernel(
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n_heads = Hq + 2 * Hkv;
     const int pos = positions[n];
-    if (R == D) {
-        for (int j = threadIdx.x; j < D / 2; j += blockDim.x) {
+    if (EXTRA || R == D) {
+        for (int j = threadIdx.x; j < (EXTRA ? R / 2 : D / 2); j += blockDim.x) {
             const float ang = (float)pos * inv_freq[j];
             cs[j] = cosf(ang);
             sn[j] = sinf(ang);
@@ -491,8 +517,13 @@ __global__ void qk_norm_rope_kvwrite_fast_kernel(
             const bool is_k = !is_q && head < Hq + Hkv;
             const bool is_v = !is_q && !is_k;
             if (!is_q && !write_kv) continue;
+            if (EXTRA && extra.bias != nullptr) {
+                const Pack<float, VPL> b = *reinterpret_cast<const Pack<float, VPL>*>(extra.bias + (size_t)head * D + lane * VPL);
+#pragma unroll
+                for (int i = 0; i < VPL; ++i) y[u][i] += b.v[i];
+            }
             const float* gain = is_q ? q_gain : (is_k ? k_gain : nullptr);
-            if (gain != nullptr) {
+            if (gain != nullptr || (EXTRA && extra.unit && !is_v)) {
                 float ss = 0.f;
 #pragma unroll
                 for (int i = 0; i < VPL; ++i) ss += y[u][i] * y[u][i];
@@ -503,7 +534,24 @@ __global__ void qk_norm_rope_kvwrite_fast_kernel(
                     y[u][i] = y[u][i] * rinv * (is_q ? gq[i] : gk[i]);
             }
             Pack<T, VPL> o;
-            if (!is_v && R == D) {
+            if (EXTRA && is_v) {
+                const size_t at = ((size_t)n * Hkv + (head - Hq - Hkv)) * D + lane * VPL;
+#pragma unroll
+                for (int i = 0; i < VPL; ++i) o.v[i] = from_float<T>(extra.value(y[u][i], at + i));
+            } else if (EXTRA && R < D) {
+                const int hl = R / 2 / VPL;              // lanes that hold the first half of the rotating dims
+                const bool first = lane < hl, second = !first && lane < 2 * hl;
+                const int mate = first ? lane + hl : second ? lane - hl : lane;
+                const int at = (first ? lane : second ? lane - hl : 0) * VPL;
+#pragma unroll
+                for (int i = 0; i < VPL; ++i) {
+                    const float partner = __shfl_sync(0xffffffffu, y[u][i], mate);
+                    float r = y[u][i];
+                    if (first) r = y[u][i] * cs[at + i] - partner * sn[at + i];
+                    if (second) r = y[u][i] * cs[at + i] + partner * sn[at + i];
+                    o.v[i] = from_float<T>(r);
+                }
+            } else if (!is_v && R == D) {
 #pragma unroll
                 for (int i = 0; i < VPL; ++i) {
                     const float partner = __shfl_xor_sync(0xffffffffu, y[u][i], 16);
@@ -532,14 +580,14 @@ __global__ void qk_norm_rope_kvwrite_fast_kernel(
 // elements, its rotation partner is lane l ^ 8), so a warp serves two heads with the
 // instructions of one.  Every shuffle is executed by all lanes whatever their heads are (the
 // two halves may hold heads of different kinds); loads and stores are predicated instead.
-template <typename T, int VPL>
+template <typename T, int VPL, bool EXTRA>
 __global__ void qk_norm_rope_kvwrite_rows_kernel(
     const T* __restrict__ qkv, const float* __restrict__ parts, int S, size_t part_stride,
     T* __restrict__ q_out, T* __restrict__ k_pool, T* __restrict__ v_pool,
     const float* __restrict__ q_gain, const float* __restrict__ k_gain,
     const float* __restrict__ inv_freq, int R, const int* __restrict__ positions,
     const int* __restrict__ token_rows, const int* __restrict__ block_table, int table_width,
-    int BS, float eps, int Hq, int Hkv, int write_kv, int heads_per_block) {
+    int BS, float eps, int Hq, int Hkv, int write_kv, int heads_per_block, QkExtra extra) {
     sb::pdl_launch_dependents();     // the next kernel may begin its prologue
     constexpr int D = 16 * VPL;
     __shared__ float cs[D / 2], sn[D / 2];
@@ -548,8 +596,8 @@ __global__ void qk_norm_rope_kvwrite_rows_kernel(
     const int sub = lane >> 4, l = lane & 15;           // which of the warp's two heads, lane within it
     const int n_heads = Hq + 2 * Hkv;
     const int pos = positions[n];
-    if (R == D) {
-        for (int j = threadIdx.x; j < D / 2; j += blockDim.x) {
+    if (EXTRA || R == D) {
+        for (int j = threadIdx.x; j < (EXTRA ? R / 2 : D / 2); j += blockDim.x) {
             const float ang = (float)pos * inv_freq[j];
             cs[j] = cosf(ang);
             sn[j] = sinf(ang);
@@ -587,6 +635,14 @@ __global__ void qk_norm_rope_kvwrite_rows_kernel(
                 for (int i = 0; i < VPL; ++i) y[i] = to_float(p.v[i]);
             }
         }
+        if (EXTRA && live && extra.bias != nullptr) {
+            const float* b = extra.bias + (size_t)head * D + l * VPL;
+#pragma unroll
+            for (int i = 0; i < VPL; i += 4) {
+                const float4 bv = *reinterpret_cast<const float4*>(b + i);
+                y[i] += bv.x; y[i + 1] += bv.y; y[i + 2] += bv.z; y[i + 3] += bv.w;
+            }
+        }
         const float* gain = is_q ? q_gain : (is_k ? k_gain : nullptr);
         float ss = 0.f;
 #pragma unroll
@@ -597,11 +653,31 @@ __global__ void qk_norm_rope_kvwrite_rows_kernel(
             const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
 #pragma unroll
             for (int i = 0; i < VPL; ++i) y[i] = y[i] * rinv * gain[l * VPL + i];
+        } else if (EXTRA && extra.unit && live && !is_v) {
+            const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
+#pragma unroll
+            for (int i = 0; i < VPL; ++i) y[i] *= rinv;
         }
         Pack<T, VPL> o;
+        if (EXTRA) {
+            const int hl = R / 2 / VPL;
+            const bool first = l < hl, second = !first && l < 2 * hl;
+            const int mate = (lane & 16) | (first ? l + hl : second ? l - hl : l);
+            const int at = (first ? l : second ? l - hl : 0) * VPL;
+            const size_t vat = ((size_t)n * Hkv + (is_v ? head - Hq - Hkv : 0)) * D + l * VPL;
+#pragma unroll
+            for (int i = 0; i < VPL; ++i) {
+                const float partner = __shfl_sync(0xffffffffu, y[i], mate);
+                float r = y[i];
+                if (is_v) { if (live) r = extra.value(y[i], vat + i); }
+                else if (first) r = y[i] * cs[at + i] - partner * sn[at + i];
+                else if (second) r = y[i] * cs[at + i] + partner * sn[at + i];
+                o.v[i] = from_float<T>(r);
+            }
+        }
         const bool rotate = !is_v && R == D;
 #pragma unroll
-        for (int i = 0; i < VPL; ++i) {
+        for (int i = 0; i < VPL && !EXTRA; ++i) {
             const float partner = __shfl_xor_sync(0xffffffffu, y[i], 8);
             const float c = cs[(l & 7) * VPL + i], s = sn[(l & 7) * VPL + i];
             const float r = l < 8 ? y[i] * c - partner * s : y[i] * c + partner * s;
@@ -624,12 +700,13 @@ static void qk_launch(const void* qkv, const float* parts, int S, size_t part_st
                       void* v_pool, const float* q_gain, const float* k_gain, const float* inv_freq,
                       int rotary_dim, const int* positions, const int* token_rows, const int* block_table,
                       int table_width, int page_size, float eps, int Hq, int Hkv, int D, int N, int write_kv,
-                      int Dv, int row_width, int neighbours, const float* bias, int sub, float magnitude,
+                      int Dv, int row_width, int neighbours, const QkExtra& extra, int sub, float magnitude,
                       int spread, cudaStream_t stream) {
     const int n_heads = Hq + 2 * Hkv;
-    const bool fast = (rotary_dim == D || rotary_dim == 0) && (D == 64 || D == 128 || D == 256) && Dv == D &&
-                      row_width == n_heads * D && !(neighbours && rotary_dim > 0) && bias == nullptr && sub == D &&
-                      magnitude == 1.0f && !spread;
+    const bool plain = (rotary_dim == D || rotary_dim == 0) && !extra.any();
+    const bool fast = (plain || rotary_dim % (D / 8) == 0) && (D == 64 || D == 128 || D == 256) && Dv == D &&
+                      row_width == n_heads * D && !(neighbours && rotary_dim > 0) && sub == D && magnitude == 1.0f &&
+                      !spread && (reinterpret_cast<uintptr_t>(extra.bias) & 15) == 0;
     // Heads per block: 4 (a head per warp) while that still fills the GPU, more for long batches.
     int hpb = 4;
     {
@@ -647,14 +724,16 @@ static void qk_launch(const void* qkv, const float* parts, int S, size_t part_st
     // Many tokens (hpb > 4): the kernel with half a warp per head (a prompt of 2,048 tokens through the 36
     // layers of the 4B shape: 20.5 -> 19.9 ms).
 #define SB_QK_FAST(VPL_) \
-    if (hpb > 4) sb::launch(qk_norm_rope_kvwrite_rows_kernel<T, 2 * VPL_>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, write_kv, hpb); \
-    else sb::launch(qk_norm_rope_kvwrite_fast_kernel<T, VPL_>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, write_kv, hpb);
+    if (hpb > 4 && plain) sb::launch(qk_norm_rope_kvwrite_rows_kernel<T, 2 * VPL_, false>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, write_kv, hpb, extra); \
+    else if (hpb > 4) sb::launch(qk_norm_rope_kvwrite_rows_kernel<T, 2 * VPL_, true>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, write_kv, hpb, extra); \
+    else if (plain) sb::launch(qk_norm_rope_kvwrite_fast_kernel<T, VPL_, false>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, write_kv, hpb, extra); \
+    else sb::launch(qk_norm_rope_kvwrite_fast_kernel<T, VPL_, true>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, write_kv, hpb, extra);
     if (fast && D == 64) { SB_QK_FAST(2) }
     else if (fast && D == 128) { SB_QK_FAST(4) }
     else if (fast) { SB_QK_FAST(8) }
 #undef SB_QK_FAST
     else sb::launch(qk_norm_rope_kvwrite_kernel<T>, dim3(grid), dim3(128), 0, stream, SB_QK_ARGS, D, write_kv, Dv,
-                    row_width, neighbours, bias, sub, magnitude, spread, hpb);
+                    row_width, neighbours, extra, sub, magnitude, spread, hpb);
 #undef SB_QK_ARGS
 }
 
@@ -667,7 +746,12 @@ extern "C" int sb_qk_norm_rope_kvwrite(const void* qkv, const float* parts, int 
                                        const int* token_rows, const int* block_table, int table_width,
                                        int page_size, float eps, int Hq, int Hkv, int D, int N,
                                        int write_kv, int dtype, int Dv, int row_width, int neighbours,
-                                       const float* bias, int sub, float magnitude, int spread, cudaStream_t stream) {
+                                       const float* bias, int sub, float magnitude, int spread, int unit, int values,
+                                       float blend, float* v_first, cudaStream_t stream) {
+    SB_REQUIRE(values >= 0 && values <= 2 && (values == 0 || (v_first != nullptr && write_kv)),
+               "qk_norm_rope: shared values (%d) need their buffer and pages to write to", values);
+    SB_REQUIRE(!unit || (q_gain == nullptr && k_gain == nullptr), "qk_norm_rope: a norm without a gain takes none");
+    const QkExtra extra{bias, unit, values, blend, v_first};
     if (sub <= 0) sub = D;
     SB_REQUIRE(D % sub == 0 && rotary_dim <= sub, "qk_norm_rope: heads of %d dims do not hold maps of %d with %d rotating",
                D, sub, rotary_dim);
@@ -686,23 +770,28 @@ extern "C" int sb_qk_norm_rope_kvwrite(const void* qkv, const float* parts, int 
     if (dtype == SB_F32)
         qk_launch<float>(qkv, parts, S, (size_t)part_stride, q_out, k_pool, v_pool, q_gain, k_gain, inv_freq,
                          rotary_dim, positions, token_rows, block_table, table_width, page_size, eps, Hq, Hkv, D, N,
-                         write_kv, Dv, row_width, neighbours, bias, sub, magnitude, spread, stream);
+                         write_kv, Dv, row_width, neighbours, extra, sub, magnitude, spread, stream);
     else if (dtype == SB_BF16)
         qk_launch<__nv_bfloat16>(qkv, parts, S, (size_t)part_stride, q_out, k_pool, v_pool, q_gain, k_gain,
                                  inv_freq, rotary_dim, positions, token_rows, block_table, table_width, page_size,
-                                 eps, Hq, Hkv, D, N, write_kv, Dv, row_width, neighbours, bias, sub, magnitude, spread, stream);
+                                 eps, Hq, Hkv, D, N, write_kv, Dv, row_width, neighbours, extra, sub, magnitude, spread, stream);
     else
         SB_REQUIRE(false, "qk_norm_rope: unknown dtype %d", dtype);
     SB_LAUNCH_CHECK();
 }
 
 // ----------------------------------------------------------------------------------------
-// SiLU*mul: out[n, f] = up * gate * sigmoid(gate).  Two layouts of the input row of 2F:
+// Gated unit: out[n, f] = up * act(gate), act silu (z * sigmoid(z)) or gelu in its tanh form.  Two layouts of the input row of 2F:
 // concatenated (gate = in[n, f], up = in[n, F + f]) or interleaved (gate = in[n, 2f],
 // up = in[n, 2f + 1]; the layout of a product with interleaved gate/up weight rows).
+__device__ __forceinline__ float gate_act(float g, int gelu) {
+    if (gelu) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+    return g / (1.0f + expf(-g));
+}
+
 template <typename T>
 __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ in, size_t total, int F,
-                                int interleaved) {
+                                int interleaved, int gelu) {
     sb::pdl_launch_dependents();     // the next kernel may begin its prologue
     sb::pdl_wait();                  // everything before this kernel is complete and visible
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total;
@@ -711,14 +800,14 @@ __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ in, s
         const int f = (int)(i - n * F);
         const float g = to_float(in[n * 2 * F + (interleaved ? 2 * f : f)]);
         const float u = to_float(in[n * 2 * F + (interleaved ? 2 * f + 1 : F + f)]);
-        out[i] = from_float<T>(u * (g / (1.0f + expf(-g))));
+        out[i] = from_float<T>(u * gate_act(g, gelu));
     }
 }
 
 // F a multiple of the 16-byte vector width: one vector of gate and one of up per thread.
 template <typename T>
 __global__ void silu_mul_vec_kernel(T* __restrict__ out, const T* __restrict__ in, size_t total_vec, int F,
-                                    int interleaved) {
+                                    int interleaved, int gelu) {
     sb::pdl_launch_dependents();     // the next kernel may begin its prologue
     sb::pdl_wait();                  // everything before this kernel is complete and visible
     constexpr int VEC = Vec16<T>::N;
@@ -736,7 +825,7 @@ __global__ void silu_mul_vec_kernel(T* __restrict__ out, const T* __restrict__ i
             for (int e = 0; e < VEC; ++e) {
                 const float gv = e < VEC / 2 ? g.get(2 * e) : u.get(2 * e - VEC);
                 const float uv = e < VEC / 2 ? g.get(2 * e + 1) : u.get(2 * e + 1 - VEC);
-                r[e] = uv * (gv / (1.0f + expf(-gv)));
+                r[e] = uv * gate_act(gv, gelu);
             }
         } else {
             g.load(in + n * 2 * F + f);
@@ -744,7 +833,7 @@ __global__ void silu_mul_vec_kernel(T* __restrict__ out, const T* __restrict__ i
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
                 const float gv = g.get(e);
-                r[e] = u.get(e) * (gv / (1.0f + expf(-gv)));
+                r[e] = u.get(e) * gate_act(gv, gelu);
             }
         }
         T* o = out + n * F + f;
@@ -762,7 +851,7 @@ __global__ void silu_mul_vec_kernel(T* __restrict__ out, const T* __restrict__ i
     }
 }
 
-extern "C" int sb_silu_mul(void* out, const void* gate_up, int N, int F, int interleaved, int dtype,
+extern "C" int sb_silu_mul(void* out, const void* gate_up, int N, int F, int interleaved, int gelu, int dtype,
                            cudaStream_t stream) {
     SB_REQUIRE(N >= 0 && F > 0, "silu_mul: bad sizes N=%d F=%d", N, F);
     if (N == 0) return 0;
@@ -774,10 +863,10 @@ extern "C" int sb_silu_mul(void* out, const void* gate_up, int N, int F, int int
         size_t blocks = (total_vec + 255) / 256;
         if (blocks > 148 * 32) blocks = 148 * 32;
         if (dtype == SB_F32)
-            sb::launch(silu_mul_vec_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, (float*)out, (const float*)gate_up, total_vec, F, interleaved);
+            sb::launch(silu_mul_vec_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, (float*)out, (const float*)gate_up, total_vec, F, interleaved, gelu);
         else if (dtype == SB_BF16)
             sb::launch(silu_mul_vec_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, stream, 
-                (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, total_vec, F, interleaved);
+                (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, total_vec, F, interleaved, gelu);
         else
             SB_REQUIRE(false, "silu_mul: unknown dtype %d", dtype);
         SB_LAUNCH_CHECK();
@@ -785,10 +874,10 @@ extern "C" int sb_silu_mul(void* out, const void* gate_up, int N, int F, int int
     size_t blocks = (total + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     if (dtype == SB_F32)
-        sb::launch(silu_mul_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, (float*)out, (const float*)gate_up, total, F, interleaved);
+        sb::launch(silu_mul_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, (float*)out, (const float*)gate_up, total, F, interleaved, gelu);
     else if (dtype == SB_BF16)
         sb::launch(silu_mul_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, stream, 
-            (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, total, F, interleaved);
+            (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, total, F, interleaved, gelu);
     else
         SB_REQUIRE(false, "silu_mul: unknown dtype %d", dtype);
     SB_LAUNCH_CHECK();

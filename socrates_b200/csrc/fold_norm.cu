@@ -7,6 +7,8 @@
 //                   residual[r] = v ;  out[m] = v / sqrt(mean(v^2) + eps) * gain    (if out)
 //                   (out with a null gain: out[m] = v, the stream itself in the model dtype, for
 //                   blocks whose branches read the stream without a norm in front)
+//                   (with norm_residual, for blocks that norm AFTER the sum: v = res_scale * residual[r] + b + ..., and
+//                   the normed row is the new residual[r] as well as out[m])
 //                   (with tanh_alpha: out[m] = tanh(alpha v) * gain + tanh_bias, nothing is averaged)
 //   normed_mean:    out[r] = scale * sum_t unit_rms(sum_s x_t[s][r]) * gain_t       (t < 2)
 //   bias_act:       out[r][f] = act(sum_s in[s][r][f] + bias[f])
@@ -36,6 +38,8 @@ struct FoldArgs {
     int write_residual;
     const float* tanh_alpha;   // [1] or null: the out rows are tanh(alpha v) * gain + tanh_bias
     const float* tanh_bias;    // [d]
+    float res_scale;           // multiplies the residual before anything is added
+    int norm_residual;         // the normed row (out may be null then) becomes the residual
 };
 
 template <typename T>
@@ -73,13 +77,24 @@ __global__ void __launch_bounds__(256) fold_rmsnorm_kernel(FoldArgs a) {
     float* res = a.residual + (size_t)r * d;
     float ss = 0.f;
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
-        float v = res[i];
+        float v = res[i] * a.res_scale;
         if (branch) v += a.branch_gain ? row[i] * binv * a.branch_gain[i] : row[i];
         if (a.add_rows) v += a.add_rows[(size_t)r * d + i];
         if (a.add_vec) v += a.add_vec[i];
         row[i] = v;
         if (a.write_residual) res[i] = v;
         ss += v * v;
+    }
+    if (a.norm_residual) {
+        const float total = block_sum(ss, scratch);
+        const float rinv = 1.0f / sqrtf(total / (float)d + a.eps);
+        T* o = (T*)a.out + (size_t)m * d;
+        for (int i = threadIdx.x; i < d; i += blockDim.x) {
+            const float y = row[i] * rinv * a.gain[i];
+            res[i] = y;
+            if (a.out != nullptr) o[i] = from_float<T>(y);
+        }
+        return;
     }
     if (a.out == nullptr) return;
     T* o = (T*)a.out + (size_t)m * d;
@@ -143,6 +158,7 @@ __global__ void __launch_bounds__(512) fold_rmsnorm_vec_kernel(FoldArgs a) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < d4; i += blockDim.x) {
         float4 v = res4[i];
+        v.x *= a.res_scale; v.y *= a.res_scale; v.z *= a.res_scale; v.w *= a.res_scale;
         if (branch) {
             float4 b = row4[i];
             if (a.branch_gain) {
@@ -163,7 +179,7 @@ __global__ void __launch_bounds__(512) fold_rmsnorm_vec_kernel(FoldArgs a) {
         if (a.write_residual) res4[i] = v;
         ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
-    if (a.out == nullptr) return;
+    if (a.out == nullptr && !a.norm_residual) return;
     const bool squash = a.tanh_alpha != nullptr, normed = a.gain != nullptr && !squash;
     const float alpha = squash ? *a.tanh_alpha : 0.f;
     const float rinv = normed ? 1.0f / sqrtf(block_sum(ss, scratch) / (float)a.d + a.eps) : 1.0f;
@@ -177,6 +193,10 @@ __global__ void __launch_bounds__(512) fold_rmsnorm_vec_kernel(FoldArgs a) {
             const float4 b = __ldg(reinterpret_cast<const float4*>(a.tanh_bias) + i);
             x0 = fmaf(tanhf(alpha * v.x), c.x, b.x); x1 = fmaf(tanhf(alpha * v.y), c.y, b.y);
             x2 = fmaf(tanhf(alpha * v.z), c.z, b.z); x3 = fmaf(tanhf(alpha * v.w), c.w, b.w);
+        }
+        if (a.norm_residual) {
+            res4[i] = make_float4(x0, x1, x2, x3);
+            if (a.out == nullptr) continue;
         }
         if constexpr (sizeof(T) == 2) {
             __nv_bfloat162 lo = __floats2bfloat162_rn(x0, x1), hi = __floats2bfloat162_rn(x2, x3);
@@ -268,7 +288,10 @@ extern "C" int sb_fold_rmsnorm(float* residual, const float* delta, int S, long 
                                const float* branch_bias, const float* branch_gain, float branch_eps,
                                const float* add_rows, const float* add_vec, const float* gain, void* out,
                                const int* row_index, int M, int d, float eps, const float* tanh_alpha,
-                               const float* tanh_bias, int out_dtype, cudaStream_t stream) {
+                               const float* tanh_bias, float res_scale, int norm_residual, int out_dtype,
+                               cudaStream_t stream) {
+    SB_REQUIRE(!norm_residual || (gain != nullptr && row_index == nullptr && tanh_alpha == nullptr),
+               "fold_rmsnorm: a normed residual needs a gain and every row");
     SB_REQUIRE(M >= 0 && d > 0 && S >= 0, "fold_rmsnorm: bad sizes M=%d d=%d S=%d", M, d, S);
     SB_REQUIRE(S == 0 || delta != nullptr, "fold_rmsnorm: S=%d partial sums but no buffer", S);
     SB_REQUIRE((tanh_alpha != nullptr) == (tanh_bias != nullptr) && (tanh_alpha == nullptr || gain != nullptr),
@@ -281,8 +304,9 @@ extern "C" int sb_fold_rmsnorm(float* residual, const float* delta, int S, long 
     a.branch_bias = branch_bias; a.branch_gain = branch_gain; a.branch_eps = branch_eps;
     a.add_rows = add_rows; a.add_vec = add_vec; a.gain = gain; a.out = out; a.row_index = row_index;
     a.d = d; a.eps = eps; a.tanh_alpha = tanh_alpha; a.tanh_bias = tanh_bias;
-    a.write_residual = row_index == nullptr &&
-                       (S > 0 || branch_bias != nullptr || add_rows != nullptr || add_vec != nullptr);
+    a.res_scale = res_scale; a.norm_residual = norm_residual;
+    a.write_residual = row_index == nullptr && !norm_residual &&
+                       (S > 0 || res_scale != 1.0f || branch_bias != nullptr || add_rows != nullptr || add_vec != nullptr);
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     const bool vec = d % 4 == 0 && delta_stride % 4 == 0 && aligned(residual) && aligned(delta) && aligned(branch_bias) &&
                      aligned(branch_gain) && aligned(add_rows) && aligned(add_vec) && aligned(gain) && aligned(tanh_bias) &&

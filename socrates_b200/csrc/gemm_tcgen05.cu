@@ -292,7 +292,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
             } else {
                 tmem_ld_wait();
             }
-            if (SWAP && EPI == 1) {
+            if (SWAP && EPI != 0) {
                 // weight rows interleave gate and up: lane pairs (even = gate_f, odd = up_f);
                 // the even lane writes C[m, f] = up * silu(gate), C has N/2 columns
                 const int n = a0 + lane_row;
@@ -303,7 +303,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
                     const float up = __shfl_xor_sync(0xffffffffu, v, 1);
                     const int m = b0 + c0 + j;
                     if ((lane & 1) == 0 && n + 1 < N && m < M)
-                        store_out<TC>(C + (size_t)m * F + (n >> 1), up * (v / (1.0f + expf(-v))));
+                        store_out<TC>(C + (size_t)m * F + (n >> 1), up * gate_act<EPI>(v));
                 }
             } else if (SWAP) {
                 const int n = a0 + lane_row;
@@ -399,7 +399,7 @@ int dispatch(const void* A, const void* W, void* C, int M, int N, int K, int spl
     *splits_out = splits;
     CUtensorMap ma, mb;
     if (M <= 64 && epi != 0 && splits != 1) {
-        sb_set_error("gemm_tcgen05: the fused SiLU*mul epilogue cannot follow a K split");
+        sb_set_error("gemm_tcgen05: the fused gated epilogue cannot follow a K split");
         return SB_ERR_ARG;
     }
     if (M <= 64) {
@@ -418,6 +418,11 @@ int dispatch(const void* A, const void* W, void* C, int M, int N, int K, int spl
             if (bn == 32) return launch<32, 5, true, TC, 1>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
             return launch<64, 4, true, TC, 1>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
         }
+        if (epi == 2) {
+            if (bn == 16) return launch<16, 6, true, TC, 2>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
+            if (bn == 32) return launch<32, 5, true, TC, 2>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
+            return launch<64, 4, true, TC, 2>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
+        }
         if (bn == 16) return launch<16, 6, true, TC>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
         if (bn == 32) return launch<32, 5, true, TC>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
         return launch<64, 4, true, TC>(ma, mb, C, M, N, K, grid, kb_per_split, status, stream);
@@ -425,7 +430,7 @@ int dispatch(const void* A, const void* W, void* C, int M, int N, int K, int spl
     if (splits == 1 && N >= 128 && variant != 4)      // the persistent kernels (gemm_tcgen05_rows.cu)
         return sb::gemm_tcgen05_many_rows(A, W, C, M, N, K, sizeof(TC) == 2 ? SB_BF16 : SB_F32, status, variant, epi, stream);
     if (epi != 0) {
-        sb_set_error("gemm_tcgen05: the fused SiLU*mul epilogue needs N >= 128 and no K split");
+        sb_set_error("gemm_tcgen05: the fused gated epilogue needs N >= 128 and no K split");
         return SB_ERR_ARG;
     }
     // variant 4: the one-tile-per-block kernel also for many rows
@@ -452,8 +457,8 @@ int dispatch(const void* A, const void* W, void* C, int M, int N, int K, int spl
 //          1256 = the pair kernel (two SMs per tile, cta_group::2) with tiles 256 x (variant - 1000);
 //          2000 = the pair kernel dealing equal shares of K blocks, float32 partial sums
 //          [parts, M, N] with *splits_io == sb_gemm_tcgen05_shares_parts(M, N, K).
-// epilogue: 0 = C[M,N]; 1 = W interleaves gate and up rows and C is [M, N/2] = up * silu(gate)
-//          (no K split; for many rows N >= 128).
+// epilogue: 0 = C[M,N]; 1 = W interleaves gate and up rows and C is [M, N/2] = up * silu(gate); 2 = the same with
+//          the tanh form of gelu (no K split; for many rows N >= 128).
 // next_weights / next_bytes: null / 0, or a 16-byte aligned range that the product after this
 //          one streams; the weight-streaming kernel (M <= 64) asks for it in L2 once its own
 //          loads are issued.  A hint: other kernels ignore it.
@@ -468,7 +473,7 @@ extern "C" int sb_gemm_tcgen05(void* C, const void* A, const void* W, int M, int
     int splits = *splits_io;
     SB_REQUIRE(splits >= 1 && splits <= 64, "gemm_tcgen05: splits=%d is outside 1..64", splits);
     SB_REQUIRE(splits == 1 || c_dtype == SB_F32, "gemm_tcgen05: partial sums of a split product are float32");
-    SB_REQUIRE(epilogue == 0 || (epilogue == 1 && N % 2 == 0), "gemm_tcgen05: bad epilogue %d for N=%d", epilogue, N);
+    SB_REQUIRE(epilogue == 0 || ((epilogue == 1 || epilogue == 2) && N % 2 == 0), "gemm_tcgen05: bad epilogue %d for N=%d", epilogue, N);
     SB_REQUIRE((M + 127) / 128 <= 65535 && (N + 63) / 64 <= 65535, "gemm_tcgen05: matrix too large");
     SB_REQUIRE(next_bytes >= 0 && (reinterpret_cast<uintptr_t>(next_weights) & 15) == 0,
                "gemm_tcgen05: the next-weights hint must be 16-byte aligned");

@@ -796,6 +796,7 @@ int many_rows(const void* A, const void* W, void* C, int M, int N, int K, int* s
         }
 #define SB_TRY(BN_) \
         if (bn == BN_) return epi == 1 ? launch_pair<BN_, pair_stages(BN_), TC, 1>(ma, mb, C, M, N, K, status, stream) \
+                            : epi == 2 ? launch_pair<BN_, pair_stages(BN_), TC, 2>(ma, mb, C, M, N, K, status, stream) \
                                        : launch_pair<BN_, pair_stages(BN_), TC, 0>(ma, mb, C, M, N, K, status, stream);
         SB_PAIR_WIDTHS(SB_TRY)
 #undef SB_TRY
@@ -814,6 +815,7 @@ int many_rows(const void* A, const void* W, void* C, int M, int N, int K, int* s
         }
 #define SB_TRY(BN_) \
         if (bn == BN_) return epi == 1 ? launch_persistent<BN_, persistent_stages(BN_), TC, 1, row_issuers(BN_, 1)>(ma, mb, C, M, N, K, status, stream) \
+                            : epi == 2 ? launch_persistent<BN_, persistent_stages(BN_), TC, 2, row_issuers(BN_, 2)>(ma, mb, C, M, N, K, status, stream) \
                                        : launch_persistent<BN_, persistent_stages(BN_), TC, 0, row_issuers(BN_, 0)>(ma, mb, C, M, N, K, status, stream);
         SB_PERSISTENT_WIDTHS(SB_TRY)
 #undef SB_TRY

@@ -9,6 +9,10 @@
 //                weights[n][e] = s_e for chosen e, else 0 ;  ids[n][k], picked[n][k] = the choices, best first
 //   router:      logits and choice in one kernel: the `top` largest of z + bias are chosen; their weights are the
 //                softmax over these only
+//                or, by scores s = sigmoid(z): the E outputs form groups of neighbours, a group counts with the sum of its
+//                two largest s, only the `keep` best groups stay, the `top` largest s there are chosen and weigh
+//                s / (their sum + 1e-20) * scale
+//   act:         all experts' units without a gate:  act[n][e*F + f] = relu(sum_s in[s][n][e*F + f])^2 * weights[n][e]
 //   glu_clamp:   all experts' gated units and the shared one's in one pass, scaled on the way out:
 //                g = min(pg, limit) ,  u = clamp(pu, -limit, limit) ,  act = g * sigmoid(alpha g) * (u + offset) * weight
 //   scale:       act[n][e*F + f] *= weights[n][e]                (all experts' activations side by side)
@@ -126,6 +130,8 @@ struct RouterArgs {
     int* ids;                  // [N, top]
     float* picked;             // [N, top]
     int N, E, K, top;
+    int sigmoid, groups, keep; // sigmoid: choose and weigh by sigmoid scores, inside the `keep` best of `groups`
+    float scale;
 };
 
 template <typename T, int TT>
@@ -183,7 +189,7 @@ __global__ void __launch_bounds__(TT == 1 ? 1024 : 256) moe_router_kernel(Router
         for (int t = 0; t < TT; ++t) {
             const float z = warp_sum(acc[t]);
             if (lane == 0) {
-                zs[t * 2 * E + e] = z + b;
+                zs[t * 2 * E + e] = a.sigmoid ? 1.0f / (1.0f + expf(-(z + b))) : z + b;
                 zs[t * 2 * E + E + e] = 0.f;
             }
         }
@@ -194,6 +200,36 @@ __global__ void __launch_bounds__(TT == 1 ? 1024 : 256) moe_router_kernel(Router
         if (n >= a.N) break;
         float *c = zs + t * 2 * E, *w = c + E;
         float best = 0.f, sum = 0.f;
+        if (a.sigmoid && a.keep < a.groups) {
+            // w serves as scratch: w[g] = the group's score, then +inf for a group that stays
+            const int per = E / a.groups;
+            for (int g = lane; g < a.groups; g += 32) {
+                float first = 0.f, second = 0.f;
+                for (int e = g * per; e < (g + 1) * per; ++e) {
+                    const float v = c[e];
+                    if (v > first) { second = first; first = v; }
+                    else if (v > second) second = v;
+                }
+                w[g] = first + second;
+            }
+            __syncwarp();
+            for (int it = 0; it < a.keep; ++it) {
+                float bv = -INFINITY;
+                int bi = 0x7fffffff;
+                for (int g = lane; g < a.groups; g += 32) {
+                    const float v = w[g];
+                    if (v != INFINITY && (v > bv || bi == 0x7fffffff)) { bv = v; bi = g; }
+                }
+                warp_argmax(bv, bi);
+                if (lane == 0 && bi < a.groups) w[bi] = INFINITY;
+                __syncwarp();
+            }
+            for (int e = lane; e < E; e += 32)
+                if (w[e / per] != INFINITY) c[e] = -INFINITY;
+            __syncwarp();
+            for (int g = lane; g < a.groups; g += 32) w[g] = 0.f;
+            __syncwarp();
+        }
         for (int k = 0; k < a.top; ++k) {
             float bv = -INFINITY;
             int bi = 0x7fffffff;
@@ -203,7 +239,7 @@ __global__ void __launch_bounds__(TT == 1 ? 1024 : 256) moe_router_kernel(Router
             }
             warp_argmax(bv, bi);
             if (k == 0) best = bv;
-            const float p = expf(bv - best);
+            const float p = a.sigmoid ? bv : expf(bv - best);
             sum += p;
             if (lane == 0 && bi < E) {
                 a.ids[(size_t)n * a.top + k] = bi;
@@ -212,7 +248,7 @@ __global__ void __launch_bounds__(TT == 1 ? 1024 : 256) moe_router_kernel(Router
             }
             __syncwarp();
         }
-        const float inv = 1.0f / sum;
+        const float inv = a.sigmoid ? a.scale / (sum + 1e-20f) : 1.0f / sum;
         for (int e = lane; e < E; e += 32) a.weights[(size_t)n * E + e] = w[e] * inv;
         for (int k = lane; k < a.top; k += 32) a.picked[(size_t)n * a.top + k] = w[a.ids[(size_t)n * a.top + k]] * inv;
     }
@@ -316,6 +352,55 @@ __global__ void __launch_bounds__(256) moe_glu_clamp_vec_kernel(MoeGluArgs a, si
 #pragma unroll
         for (int j = 0; j < VEC; ++j) y[j] = from_float<T>(glu_clamped(g[j], u[j], limit, a.alpha, a.offset) * w);
         *reinterpret_cast<uint4*>(out) = *reinterpret_cast<const uint4*>(y);
+    }
+}
+
+// Units without a gate: relu squared, scaled.  VEC = 1 serves any shape; with VEC the 16-byte vector (F a multiple of
+// it) a thread takes one vector, whose elements share their expert.  An expert that was not chosen is not read.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) moe_act_kernel(MoeGluArgs a, size_t items) {
+    sb::pdl_launch_dependents();
+    sb::pdl_wait();
+    const int per_row = a.W / VEC;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < items; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t n = i / per_row;
+        const int f = (int)(i - n * per_row) * VEC;
+        const float w = a.weights[n * a.E_total + f / a.F];
+        T* out = (T*)a.out + n * a.W + f;
+        float z[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) z[j] = 0.f;
+        if (w != 0.f) {
+            if (a.parts) {
+                for (int s = 0; s < a.S; ++s) {
+                    const float* p = a.parts + s * a.part_stride + n * a.W + f;
+                    if constexpr (VEC == 1) {
+                        z[0] += *p;
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < VEC; j += 4) {
+                            const float4 x = *reinterpret_cast<const float4*>(p + j);
+                            z[j] += x.x; z[j + 1] += x.y; z[j + 2] += x.z; z[j + 3] += x.w;
+                        }
+                    }
+                }
+            } else if constexpr (VEC == 1) {
+                z[0] = to_float(((const T*)a.in)[n * a.W + f]);
+            } else {
+                Vec16<T> v;
+                v.load((const T*)a.in + n * a.W + f);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) z[j] = v.get(j);
+            }
+        }
+        alignas(16) T y[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+            const float p = fmaxf(z[j], 0.f);
+            y[j] = from_float<T>(p * p * w);
+        }
+        if constexpr (VEC == 1) *out = y[0];
+        else *reinterpret_cast<uint4*>(out) = *reinterpret_cast<const uint4*>(y);
     }
 }
 
@@ -462,7 +547,11 @@ extern "C" int sb_moe_route(const float* logits, const float* correction, float*
 
 // weights float32 [N, E]; ids int32 and picked float32 [N, top].
 extern "C" int sb_moe_router(const void* x, const float* router, const float* bias, float* weights, int* ids, float* picked,
-                             int N, int E, int K, int top, int dtype, cudaStream_t stream) {
+                             int N, int E, int K, int top, int sigmoid, int groups, int keep, float scale, int dtype,
+                             cudaStream_t stream) {
+    SB_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && (sigmoid || groups == 1),
+               "moe_router: %d outputs in %d groups of which %d stay", E, groups, keep);
+    SB_REQUIRE(top <= keep * (E / groups), "moe_router: %d choices from %d open experts", top, keep * (E / groups));
     SB_REQUIRE(N >= 0 && E > 0 && K > 0 && top >= 1 && top <= E, "moe_router: bad sizes N=%d E=%d K=%d top=%d", N, E, K, top);
     const int Kp = (K + 127) / 128 * 128;
     auto need = [&](int tt) { return (size_t)tt * (Kp + 2 * E) * sizeof(float); };
@@ -471,7 +560,7 @@ extern "C" int sb_moe_router(const void* x, const float* router, const float* bi
     if (N == 0) return 0;
     RouterArgs a;
     a.x = x; a.router = router; a.bias = bias; a.weights = weights; a.ids = ids; a.picked = picked; a.N = N; a.E = E; a.K = K;
-    a.top = top;
+    a.top = top; a.sigmoid = sigmoid; a.groups = groups; a.keep = keep; a.scale = scale;
     const bool many = N >= 512 && need(8) <= 100 * 1024;      // many tokens: a router row fetched once serves eight
     if (dtype == SB_F32) { if (many) launch_router<float, 8>(a, need(8), stream); else launch_router<float, 1>(a, need(1), stream); }
     else { if (many) launch_router<__nv_bfloat16, 8>(a, need(8), stream); else launch_router<__nv_bfloat16, 1>(a, need(1), stream); }
@@ -505,6 +594,33 @@ extern "C" int sb_moe_glu_clamp(void* out, const void* in, const float* parts, i
         else sb::launch(moe_glu_clamp_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, a, items);
     } else {
         SB_REQUIRE(false, "moe_glu_clamp: unknown dtype %d", dtype);
+    }
+    SB_LAUNCH_CHECK();
+}
+
+// in [N, experts * F] in the model dtype (or parts float32 [S, N, experts * F]); weights float32 [N, E_total].
+extern "C" int sb_moe_act(void* out, const void* in, const float* parts, int S, long long part_stride, const float* weights,
+                          int N, int E_total, int experts, int F, int dtype, cudaStream_t stream) {
+    SB_REQUIRE(N >= 0 && experts > 0 && experts <= E_total && F > 0, "moe_act: bad sizes N=%d experts=%d/%d F=%d", N,
+               experts, E_total, F);
+    SB_REQUIRE((in != nullptr) != (parts != nullptr), "moe_act: one input, a matrix or partial sums");
+    SB_REQUIRE(dtype == SB_F32 || dtype == SB_BF16, "moe_act: unknown dtype %d", dtype);
+    if (N == 0) return 0;
+    MoeGluArgs a = {};
+    a.in = in; a.parts = parts; a.S = S; a.part_stride = (size_t)part_stride; a.weights = weights; a.out = out;
+    a.W = experts * F; a.E_total = E_total; a.experts = experts; a.F = F;
+    const size_t total = (size_t)N * a.W;
+    const int vec = dtype == SB_BF16 ? 8 : 4;
+    const bool wide = F % vec == 0 && part_stride % 4 == 0 &&
+                      ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(parts) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const size_t items = wide ? total / vec : total;
+    const dim3 blocks((int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16));
+    if (dtype == SB_F32) {
+        if (wide) sb::launch(moe_act_kernel<float, 4>, blocks, dim3(256), 0, stream, a, items);
+        else sb::launch(moe_act_kernel<float, 1>, blocks, dim3(256), 0, stream, a, items);
+    } else {
+        if (wide) sb::launch(moe_act_kernel<__nv_bfloat16, 8>, blocks, dim3(256), 0, stream, a, items);
+        else sb::launch(moe_act_kernel<__nv_bfloat16, 1>, blocks, dim3(256), 0, stream, a, items);
     }
     SB_LAUNCH_CHECK();
 }

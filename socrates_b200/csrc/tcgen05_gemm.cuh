@@ -174,10 +174,21 @@ __device__ __forceinline__ void drain_tile_f32_staged(uint32_t taddr, float* __r
     }
 }
 
+// What the gated epilogues apply to the gate: EPI 1 silu, 2 gelu.
+template <int EPI> __device__ __forceinline__ float gate_act(float g) {
+    if constexpr (EPI == 2) {
+        // 0.5 g (1 + tanh(y)) = g * sigmoid(2 y),  y = sqrt(2 / pi) (g + 0.044715 g^3)
+        const float y2 = 2.0f * 0.7978845608028654f * fmaf(0.044715f * g * g, g, g);
+        return g / (1.0f + expf(-y2));
+    }
+    return g / (1.0f + expf(-g));
+}
+
 // One thread's row of a finished accumulator tile, BN columns from tensor memory at `taddr`,
 // to row m of C (columns b0 ..).  Called by whole warps: the loads are warp-wide.
 //   EPI = 0: C[m, n] = acc
 //   EPI = 1: columns interleave gate and up; C[m, f] = up * silu(gate), C has N/2 columns.
+//   EPI = 2: the same with gelu (tanh form) in place of silu.
 //   ADD > 0: a second accumulator ADD columns further on is added to the first.
 template <int BN, typename TC, int EPI, int ADD = 0>
 __device__ __forceinline__ void drain_tile(uint32_t taddr, TC* __restrict__ C, int M, int N, int m, int b0) {
@@ -195,7 +206,7 @@ __device__ __forceinline__ void drain_tile(uint32_t taddr, TC* __restrict__ C, i
             tmem_ld_wait();
         }
         if (m >= M) continue;
-        if (EPI == 1) {
+        if (EPI != 0) {
             // columns come in (gate, up) pairs: 16 accumulator columns -> 8 outputs
             const int f0 = (b0 + c0) >> 1, F = N >> 1;
             TC* row = C + (size_t)m * F + f0;
@@ -203,7 +214,7 @@ __device__ __forceinline__ void drain_tile(uint32_t taddr, TC* __restrict__ C, i
 #pragma unroll
             for (int q = 0; q < 8; ++q) {
                 const float g = __uint_as_float(r[2 * q]), u = __uint_as_float(r[2 * q + 1]);
-                o[q] = u * (g / (1.0f + expf(-g)));
+                o[q] = u * gate_act<EPI>(g);
             }
             if (f0 + 8 <= F && ((reinterpret_cast<uintptr_t>(row) & 15) == 0) && sizeof(TC) == 2) {
                 uint32_t pk[4];

@@ -198,13 +198,13 @@ class StepContext:
         return parts if shares_cost < 0.9 * whole_cost else 0
 
     def can_fuse_silu_mul(self, M: int, w: torch.Tensor, x_dtype: torch.dtype) -> bool:
-        """Whether the product with an interleaved gate/up matrix can apply SiLU*mul in its
+        """Whether the product with an interleaved gate/up matrix can apply the gated unit (SiLU or gelu) in its
         epilogue (the tensor-core kernels do, for few rows and for many)."""
         return self.uses_tensor_cores(x_dtype, w) and w.shape[0] % 2 == 0 and (M <= 64 or w.shape[0] >= 128)
 
     def gemm(self, out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, epilogue: int = 0) -> None:
-        """out = x w^T; out is [M, N] or float32 partial sums [S, M, N]; with epilogue 1 (see
-        can_fuse_silu_mul) out is [M, N/2] = up * silu(gate) of interleaved columns."""
+        """out = x w^T; out is [M, N] or float32 partial sums [S, M, N]; with epilogue 1 or 2 (see
+        can_fuse_silu_mul) out is [M, N/2] = up * silu(gate) or up * gelu(gate) of interleaved columns."""
         S = out.shape[0] if out.dim() == 3 else 1
         if self.uses_tensor_cores(x.dtype, w):
             M = x.shape[0]

@@ -30,8 +30,8 @@ _SIGNATURES = {
     "sb_set_dependent_launch": [I],
     "sb_embed": [P, P, P, I, I, I, I, P, F, P],
     "sb_add_rmsnorm": [P, P, I, LL, P, P, P, I, I, F, I, P],
-    "sb_qk_norm_rope_kvwrite": [P, P, I, LL, P, P, P, P, P, P, I, P, P, P, I, I, F, I, I, I, I, I, I, I, I, I, P, I, F, I, P],
-    "sb_silu_mul": [P, P, I, I, I, I, P],
+    "sb_qk_norm_rope_kvwrite": [P, P, I, LL, P, P, P, P, P, P, I, P, P, P, I, I, F, I, I, I, I, I, I, I, I, I, P, I, F, I, I, I, F, P, P],
+    "sb_silu_mul": [P, P, I, I, I, I, I, P],
     "sb_sample": [P, P, P, P, P, I, I, P, P],
     "sb_sample_slices": [I],
     "sb_gemm_simt": [P, P, P, I, I, I, I, I, I, I, P],
@@ -41,14 +41,14 @@ _SIGNATURES = {
     "sb_gemm_tcgen05_shares_parts": [I, I, I],
     "sb_attention_mma_supports": [I, I, I, I, I],
     "sb_attention_prefill_mma": [P, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P],
-    "sb_attention_decode_mma": [P, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, P],
+    "sb_attention_decode_mma": [P, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, F, P, I, P],
     "sb_attention_decode_mma_blocks_per_sm": [I, I],
     "sb_attention_decode_mma_kernels": [I],
     "sb_attention_decode_stream_supports": [I, I, I, I],
     "sb_attention_decode_stream": [P, P, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "sb_attention_tcgen05_supports": [I, I, I, I],
-    "sb_attention_prefill_tcgen05": [P, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, P, P, LL, I, I, F, I, P, P],
-    "sb_fold_rmsnorm": [P, P, I, LL, P, P, F, P, P, P, P, P, I, I, F, P, P, I, P],
+    "sb_attention_prefill_tcgen05": [P, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, P, P, LL, I, I, F, I, P, F, P, I, P],
+    "sb_fold_rmsnorm": [P, P, I, LL, P, P, F, P, P, P, P, P, I, I, F, P, P, F, I, I, P],
     "sb_normed_mean": [P, P, I, LL, P, P, I, LL, P, I, I, F, F, P],
     "sb_bias_act": [P, P, P, I, LL, P, I, I, I, I, P],
     "sb_short_conv": [P, LL, P, P, P, I, P, I, I, I, P, P, P, I, I, I, P, P, P, P, P, P, P, I, P],
@@ -63,7 +63,7 @@ _SIGNATURES = {
     "sb_moe_route": [P, P, P, P, P, I, I, I, I, I, P],
     "sb_moe_scale": [P, P, I, I, I, I, I, P],
     "sb_moe_passthrough": [P, P, P, I, I, I, I, I, P],
-    "sb_attention_bias_tile": [P, P, P, P, P, I, P, P, P, I, P, LL, P, I, I, I, I, I, I, I, I, F, F, I, I, I, F, P],
+    "sb_attention_bias_tile": [P, P, P, P, P, I, P, P, P, I, P, LL, P, I, I, I, I, I, I, I, I, F, F, I, I, I, F, P, I, P],
     "sb_softcap": [P, LL, F, P],
     "sb_diff_combine": [P, P, I, I, I, F, F, F, I, P],
     "sb_moe_table": [P, P, P, P, I, I, I, I, P],
@@ -82,7 +82,8 @@ _SIGNATURES = {
     "sb_linear_recurrence": [P] + [P, I, LL, LL, I] * 4 + [P, P, P, I, I, P, P, P, I, I, I, I, I, I, I, P, P, I, P],
     "sb_norm_gate": [P, P, P, I, LL, LL, I, P, I, I, I, F, I, I, P],
     "sb_token_shift_mix": [P, P, P, P, P, I, I, I, I, P],
-    "sb_moe_router": [P, P, P, P, P, P, I, I, I, I, I, P],
+    "sb_moe_router": [P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
+    "sb_moe_act": [P, P, P, I, LL, P, I, I, I, I, I, P],
     "sb_attention_latent_supports": [I, I, I],
     "sb_attention_latent": [P, P, P, P, I, P, P, P, P, P, I, P, LL, I, I, I, I, I, I, F, I, I, P, P, P],
     "sb_moe_glu_clamp": [P, P, P, I, LL, P, I, I, I, I, I, F, F, F, F, I, P],
@@ -92,7 +93,7 @@ _SIGNATURES = {
     "sb_attention_talk_tile": [I, I, I, I],
     "sb_attention_talk_dense": [I, P, P, P, P, P, P, P, P, P, P, P, P, LL, P, I, I, I, I, I, I, I, I, I, I, I, F, P],
     "sb_attention_talk": [P, P, P, P, P, I, P, P, P, I, P, P, LL, I, I, I, I, I, I, I, F, I, I, P, P, I, P],
-    "sb_attention_bias": [P, P, P, P, P, I, P, P, P, LL, P, I, I, I, I, I, I, I, I, F, F, I, P, P, I, I, I, F, P],
+    "sb_attention_bias": [P, P, P, P, P, I, P, P, P, LL, P, I, I, I, I, I, I, I, I, F, F, I, P, P, I, I, I, F, P, I, P],
 }
 
 

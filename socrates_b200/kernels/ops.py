@@ -125,7 +125,9 @@ def qk_norm_rope_kvwrite(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optiona
                          eps: float, num_heads: int, num_kv_heads: int, head_dim: int,
                          value_dim: Optional[int] = None, row_width: Optional[int] = None,
                          neighbours: bool = False, bias: Optional[torch.Tensor] = None,
-                         map_dim: Optional[int] = None, magnitude: float = 1.0, spread_maps: bool = False) -> None:
+                         map_dim: Optional[int] = None, magnitude: float = 1.0, spread_maps: bool = False,
+                         unit_norm: bool = False, values: Optional[str] = None, blend: float = 0.0,
+                         v_first: Optional[torch.Tensor] = None) -> None:
     """Per-head norm, rotation and paged KV write for N tokens.
 
     qkv [N, (Hq+2Hkv)*D] in the model dtype, or float32 [S, N, (Hq+2Hkv)*D] partial sums
@@ -139,6 +141,8 @@ def qk_norm_rope_kvwrite(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optiona
     rotates its own first rotary_dim dims.  `magnitude` multiplies every cosine and sine.
     `spread_maps`: q_out is [N, Hq * maps, head_dim], a row per (head, map) that holds the map's dims in
     their place and zeros elsewhere, so that a dot product with a whole key row gives that map's score.
+    `unit_norm`: q and k are normed without a gain.  `values`: what `v_first` (float32 [N, Hkv*Dv]) is for:
+    "keep": this layer's values are left there too; "blend": the pages get (1 - blend) * own + blend * v_first.
     """
     Hq, Hkv, D = num_heads, num_kv_heads, head_dim
     Dv = D if value_dim is None else int(value_dim)
@@ -170,6 +174,9 @@ def qk_norm_rope_kvwrite(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optiona
             _want(g, nm, torch.float32, (D,))
     if bias is not None:
         _want(bias, "bias", torch.float32, (width,))
+    mode = {None: 0, "keep": 1, "blend": 2}[values]
+    if mode:
+        _want(v_first, "v_first", torch.float32, (N, Hkv * Dv))
     sub = D if map_dim is None else int(map_dim)
     if sub < 1 or D % sub or rotary_dim > sub:
         raise KernelError(f"heads of {D} dims do not hold maps of {sub} dims with {rotary_dim} rotating")
@@ -179,18 +186,22 @@ def qk_norm_rope_kvwrite(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optiona
         N * width, _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(q_gain), _ptr(k_gain), _ptr(inv_freq),
         rotary_dim, _ptr(positions), _ptr(token_rows), _ptr(block_table), block_table.shape[1],
         page_size, float(eps), Hq, Hkv, D, N, int(write_kv), _code(q_out.dtype), Dv, width, int(neighbours),
-        _ptr(bias), sub, float(magnitude), int(bool(spread_maps)), _stream()), "qk_norm_rope_kvwrite")
+        _ptr(bias), sub, float(magnitude), int(bool(spread_maps)), int(bool(unit_norm)), mode, float(blend),
+        _ptr(v_first) if mode else None, _stream()), "qk_norm_rope_kvwrite")
 
 
-def silu_mul(out: torch.Tensor, gate_up: torch.Tensor, interleaved: bool = False) -> None:
-    """out[n, f] = up * silu(gate) with gate = gate_up[n, f], up = gate_up[n, F + f], or, when
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}        # what a gated unit may apply to its gate; the products' epilogue is 1 + this
+
+
+def silu_mul(out: torch.Tensor, gate_up: torch.Tensor, interleaved: bool = False, act: str = "silu") -> None:
+    """out[n, f] = up * act(gate) (silu, or the tanh form of gelu) with gate = gate_up[n, f], up = gate_up[n, F + f], or, when
     `interleaved`, gate = gate_up[n, 2f], up = gate_up[n, 2f + 1]."""
     N, F2 = gate_up.shape
     _want(gate_up, "gate_up")
     _want(out, "out", gate_up.dtype, (N, F2 // 2))
     lib = library()
-    check(lib, lib.sb_silu_mul(_ptr(out), _ptr(gate_up), N, F2 // 2, int(interleaved), _code(out.dtype), _stream()),
-          "silu_mul")
+    check(lib, lib.sb_silu_mul(_ptr(out), _ptr(gate_up), N, F2 // 2, int(interleaved), GATE_ACTIVATIONS[act], _code(out.dtype),
+                               _stream()), "silu_mul")
 
 
 def sample_scratch_size(M: int, V: int) -> int:
@@ -315,7 +326,7 @@ def gemm_tcgen05(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, status: to
     if out.dim() == 2:
         if S != 1:
             raise KernelError("a split product needs a float32 [S, M, N] output")
-        _want(out, "out", None, (M, N // 2 if epilogue == 1 else N))
+        _want(out, "out", None, (M, N // 2 if epilogue else N))
     else:
         _want(out, "out", torch.float32, (S, M, N))
     lib = library()
@@ -374,12 +385,14 @@ def attention_decode_mma(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tenso
                          block_table: torch.Tensor, token_rows: torch.Tensor, positions: torch.Tensor,
                          num_heads: int, scale: float, window: int = 0, num_partitions: int = 1,
                          part_o: Optional[torch.Tensor] = None,
-                         part_ml: Optional[torch.Tensor] = None, variant: int = 0) -> None:
+                         part_ml: Optional[torch.Tensor] = None, variant: int = 0, softcap: float = 0.0,
+                         slopes: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """Paged attention of single decode tokens on the tensor cores (bfloat16), the keys
     of each token cut into `num_partitions` parts; arguments as `attention_simt`.
     `variant` picks the kernel's (warps, stages); 0 is the default.  2 to 4 partitions are
     merged inside the kernel (a thread-block cluster per token and KV head), more by a
-    reduce kernel through the scratch buffers.
+    reduce kernel through the scratch buffers.  `softcap` (0: none): s = c * tanh(s / c); `slopes` float32
+    [Hq]: a key loses slope * distance; `chunk` > 0: only keys of the query's own chunk of so many positions.
 
     The kernel reads the block table, rows, positions and the keys and values below each
     position before it waits for the kernel that precedes it on the stream: those must be
@@ -403,7 +416,8 @@ def attention_decode_mma(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tenso
     check(lib, lib.sb_attention_decode_mma(
         _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table),
         block_table.shape[1], _ptr(token_rows), _ptr(positions), N, Hq, Hkv, D, BS, int(window),
-        float(scale), num_partitions, int(variant), _stream()), "attention_decode_mma",
+        float(scale), num_partitions, int(variant), float(softcap), _slopes(slopes, Hq), int(chunk), _stream()),
+        "attention_decode_mma",
         kernels=lib.sb_attention_decode_mma_kernels(num_partitions))
 
 
@@ -469,12 +483,14 @@ def attention_prefill_tcgen05(out: torch.Tensor, q: torch.Tensor, k_pool: torch.
                               seq_first_pos: torch.Tensor, num_heads: int, scale: float, status: torch.Tensor,
                               window: int = 0, gate: Optional[torch.Tensor] = None, gate_per_dim: bool = False,
                               sink: Optional[float] = None, keep_first: int = 0,
-                              out_float: Optional[torch.Tensor] = None) -> None:
+                              out_float: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                              slopes: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """Paged causal attention of prompt portions on tcgen05 (scores and P.V in tensor
     memory, pages brought in by TMA).  Arguments as `attention_prefill_mma`, plus the int32
     status word that receives a non-zero code if a bounded wait inside the kernel gave up.
     `keep_first`: a window also sees the first so many keys of its row.  `out_float` (float32
-    [N, Hq*D]): the rows go there unrounded instead of to `out` (which may then be None)."""
+    [N, Hq*D]): the rows go there unrounded instead of to `out` (which may then be None).
+    `softcap`, `slopes`, `chunk` as in `attention_decode_mma`."""
     N = q.shape[0]
     pages, Hkv, BS, D = k_pool.shape
     R = seq_rows.numel()
@@ -500,7 +516,8 @@ def attention_prefill_tcgen05(out: torch.Tensor, q: torch.Tensor, k_pool: torch.
         _ptr(out), _ptr(q), _ptr(k_pool), _ptr(v_pool), pages, _ptr(block_table), block_table.shape[1],
         _ptr(seq_starts), _ptr(seq_rows), _ptr(seq_first_pos), R, N, num_heads, Hkv, D, BS, int(window),
         float(scale), _ptr(status), _ptr(gate), gate_stride, int(gate_per_dim), int(sink is not None),
-        float(sink or 0.0), int(keep_first), _ptr(out_float), _stream()), "attention_prefill_tcgen05")
+        float(sink or 0.0), int(keep_first), _ptr(out_float), float(softcap), _slopes(slopes, num_heads), int(chunk),
+        _stream()), "attention_prefill_tcgen05")
 
 
 # ---------------------------------------------------------------------------------------------
@@ -514,7 +531,7 @@ def fold_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: Op
                  branch_bias: Optional[torch.Tensor] = None, branch_gain: Optional[torch.Tensor] = None,
                  branch_eps: float = 0.0, add_rows: Optional[torch.Tensor] = None,
                  add_vec: Optional[torch.Tensor] = None, tanh_alpha: Optional[torch.Tensor] = None,
-                 tanh_bias: Optional[torch.Tensor] = None) -> None:
+                 tanh_bias: Optional[torch.Tensor] = None, res_scale: float = 1.0, norm_residual: bool = False) -> None:
     """b = sum(delta, 0) + branch_bias; with `branch_gain` b = b / sqrt(mean(b^2) + branch_eps) * branch_gain;
     residual += b + add_rows + add_vec; out = residual / sqrt(mean(residual^2) + eps) * gain
     (gain None with an out: out = residual, rounded to out's dtype; with `tanh_alpha`, float32 of one element,
@@ -523,6 +540,8 @@ def fold_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: Op
     residual float32 [N, d]; delta float32 [S, N, d] or None; the gains, the bias and add_vec float32 [d];
     add_rows float32 [N, d]; out [M, d] in float32 or bfloat16, or None (only the residual moves on).  With
     `row_index` only the named rows are computed and the residual is left as it is.
+    `res_scale` multiplies the residual before anything is added to it.  `norm_residual` (blocks that norm after
+    the sum): the normed row is the new residual; `out`, if given, gets it in its own dtype.
     """
     N, d = residual.shape
     _want(residual, "residual", torch.float32)
@@ -553,7 +572,8 @@ def fold_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: Op
     lib = library()
     check(lib, lib.sb_fold_rmsnorm(_ptr(residual), _ptr(delta), S, stride, _ptr(branch_bias), _ptr(branch_gain),
                                    float(branch_eps), _ptr(add_rows), _ptr(add_vec), _ptr(gain), _ptr(out),
-                                   _ptr(row_index), M, d, float(eps), _ptr(tanh_alpha), _ptr(tanh_bias), code, _stream()),
+                                   _ptr(row_index), M, d, float(eps), _ptr(tanh_alpha), _ptr(tanh_bias), float(res_scale),
+                                   int(bool(norm_residual)), code, _stream()),
           "fold_rmsnorm")
 
 
@@ -761,13 +781,20 @@ def _gate_stride(gate: Optional[torch.Tensor], q: torch.Tensor, N: int, columns:
     return gate.stride(0)
 
 
+def _slopes(slopes: Optional[torch.Tensor], Hq: int):
+    if slopes is None:
+        return None
+    _want(slopes, "slopes", torch.float32, (Hq,))
+    return _ptr(slopes)
+
+
 def attention_bias(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                    block_table: torch.Tensor, token_rows: torch.Tensor, positions: torch.Tensor, num_heads: int,
                    scale: float, window: int = 0, softcap: float = 0.0,
                    dist_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                    num_partitions: int = 1, part_o: Optional[torch.Tensor] = None,
                    part_ml: Optional[torch.Tensor] = None, gate_per_dim: bool = False,
-                   sink: Optional[float] = None) -> None:
+                   sink: Optional[float] = None, slopes: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """Paged causal attention, one query per token, with scores capped by softcap * tanh(s / softcap)
     (0: no cap), a float32 bias table [Hq, L] by distance (distances past L-1 use the last entry) and a
     sigmoid gate per head (gate [N, >= Hq], head h at column h).  Keys and values may have different head
@@ -775,7 +802,8 @@ def attention_bias(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tensor, v_p
     `gate_per_dim`: the gate is [N, >= Hq*Dv], one per head and value dim (column h*Dv + d).  `sink`: a score
     whose exponential joins the softmax denominator without a value (0.0: "one added to the denominator").
     With `num_partitions` > 1 every token's visible keys are cut into that many equal shares, one block
-    each, merged by a second kernel through the float32 scratch part_o (N*Hq*NP*Dv) and part_ml (N*Hq*NP*2)."""
+    each, merged by a second kernel through the float32 scratch part_o (N*Hq*NP*Dv) and part_ml (N*Hq*NP*2).
+    `slopes` and `chunk` as in `attention_decode_mma`."""
     N = q.shape[0]
     pages, Hkv, BS, Dk = k_pool.shape
     Dv = v_pool.shape[3]
@@ -805,7 +833,7 @@ def attention_bias(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tensor, v_p
                                      _ptr(dist_bias), L, N, Hq, Hkv, Dk, Dv, BS, int(window), float(scale),
                                      float(softcap), int(num_partitions), _ptr(part_o), _ptr(part_ml),
                                      _code(q.dtype), int(gate_per_dim), int(sink is not None),
-                                     float(sink or 0.0), _stream()), "attention_bias",
+                                     float(sink or 0.0), _slopes(slopes, Hq), int(chunk), _stream()), "attention_bias",
           kernels=2 if num_partitions > 1 else 1)
 
 
@@ -821,7 +849,8 @@ def attention_bias_tile(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tensor
                         seq_first_pos: torch.Tensor, num_heads: int, scale: float, window: int = 0,
                         softcap: float = 0.0, dist_bias: Optional[torch.Tensor] = None,
                         gate: Optional[torch.Tensor] = None, gate_per_dim: bool = False,
-                        sink: Optional[float] = None) -> None:
+                        sink: Optional[float] = None, slopes: Optional[torch.Tensor] = None,
+                        chunk: int = 0) -> None:
     """`attention_bias` for prompt portions: request r brings tokens seq_starts[r] .. seq_starts[r+1]-1 at
     positions seq_first_pos[r], +1, ... of cache row seq_rows[r]; a block serves a tile of consecutive tokens
     of one request, so a key or value row fetched once serves all of them.  The same arithmetic in float32."""
@@ -850,8 +879,8 @@ def attention_bias_tile(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tensor
                                           block_table.shape[1], _ptr(seq_starts), _ptr(seq_rows), _ptr(seq_first_pos),
                                           R, _ptr(gate), gate_stride, _ptr(dist_bias), L, N, Hq, Hkv, Dk, Dv, BS,
                                           int(window), float(scale), float(softcap), _code(q.dtype),
-                                          int(gate_per_dim), int(sink is not None), float(sink or 0.0), _stream()),
-          "attention_bias_tile")
+                                          int(gate_per_dim), int(sink is not None), float(sink or 0.0), _slopes(slopes, Hq),
+                                          int(chunk), _stream()), "attention_bias_tile")
 
 
 # Gated delta rule and the routing of a mixture of experts.
@@ -1532,10 +1561,13 @@ def token_shift_mix(out: torch.Tensor, x: torch.Tensor, mu: torch.Tensor, last: 
 
 
 def moe_router(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], weights: torch.Tensor,
-               ids: torch.Tensor, picked: torch.Tensor, top: int) -> None:
+               ids: torch.Tensor, picked: torch.Tensor, top: int, sigmoid: bool = False, groups: int = 1,
+               keep: int = 1, scale: float = 1.0) -> None:
     """Logits z = x [N, K] @ router [E, K]^T + bias (float32 weights and sums, made in the same order whatever else the
     step holds) and the choice by them: weights float32 [N, E] gets the softmax over the `top` largest logits at their
-    places and 0 elsewhere, ids int32 / picked float32 [N, top] the choices best first."""
+    places and 0 elsewhere, ids int32 / picked float32 [N, top] the choices best first.
+    `sigmoid`: scores s = sigmoid(z) choose and weigh: of `groups` equal groups of neighbours the `keep` best stay (a
+    group's score is the sum of its two largest s), the `top` largest s there get s / (their sum + 1e-20) * scale."""
     N, K = x.shape
     E = router.shape[0]
     _want(x, "x")
@@ -1547,7 +1579,28 @@ def moe_router(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tenso
     _want(picked, "picked", torch.float32, (N, top))
     lib = library()
     check(lib, lib.sb_moe_router(_ptr(x), _ptr(router), _ptr(bias), _ptr(weights), _ptr(ids), _ptr(picked), N, E, K,
-                                 int(top), _code(x.dtype), _stream()), "moe_router")
+                                 int(top), int(bool(sigmoid)), int(groups), int(keep), float(scale), _code(x.dtype),
+                                 _stream()), "moe_router")
+
+
+def moe_act(out: torch.Tensor, x: torch.Tensor, weights: torch.Tensor, experts: int, inter: int) -> None:
+    """All experts' units without a gate side by side, relu(x)^2 times the token's weight for the expert (0: not
+    computed): out [N, experts * inter]; x the same in out's dtype, or float32 partial sums [S, N, experts * inter];
+    weights float32 [N, >= experts]."""
+    N, W = out.shape
+    _want(out, "out")
+    parts = x.dim() == 3
+    if parts:
+        _want(x, "x partial sums", torch.float32, (x.shape[0], N, W))
+    else:
+        _want(x, "x", out.dtype, (N, W))
+    _want(weights, "weights", torch.float32)
+    if weights.shape[0] != N or weights.shape[1] < experts or W != experts * inter:
+        raise KernelError(f"weights {tuple(weights.shape)} do not fit {experts} experts of {inter} in {W} columns")
+    lib = library()
+    check(lib, lib.sb_moe_act(_ptr(out), None if parts else _ptr(x), _ptr(x) if parts else None,
+                              x.shape[0] if parts else 0, N * W, _ptr(weights), N, weights.shape[1], int(experts),
+                              int(inter), _code(out.dtype), _stream()), "moe_act")
 
 
 def moe_glu_clamp(out: torch.Tensor, x: torch.Tensor, weights: torch.Tensor, experts: int, inter: int, limit: float,

@@ -111,6 +111,8 @@ class ResidualStream:
     def __init__(self, residual: torch.Tensor):
         self.residual = residual
         self.pending: Optional[Branch] = None
+        # The residual as rows in the model dtype, kept by blocks that norm the stream itself.
+        self.rows: Optional[torch.Tensor] = None
         # What else joins the residual at the next fold: float32 rows [N, d] and a vector [d].
         self.add_rows: Optional[torch.Tensor] = None
         self.add_vec: Optional[torch.Tensor] = None

@@ -250,3 +250,42 @@ class BranchNormBlock(SandwichBlock):
 
 
 register_part("arrangement", "branch_norm", lambda layer_spec, name="": BranchNormBlock(layer_spec))
+
+
+class PostNormBlock:
+    """A block that norms AFTER the sum: x = norm_1(a x + mixer(x)); x = norm_2(a x + feed_forward(x)), with one
+    constant `a` (the layer's `residual_scale`) on the stream.  Mixer and feed-forward read the stream itself.  A layer
+    without a feed-forward has one norm.
+
+    The scaled sum and the norm are one kernel: it reads the branch's partial sums and the float32 residual, writes the
+    normed row back as the new residual and, in the bfloat16 engine, its rounding beside it for the next part to read
+    (`stream.rows`; the float32 engine reads the residual in place).  Nothing is left pending between layers."""
+
+    def __init__(self, layer_spec):
+        want = 2 if layer_spec.feed_forward is not None else 1
+        if len(layer_spec.norms) != want:
+            raise ValueError(f"a post_norm block with{'' if want == 2 else 'out'} a feed-forward has {want} norm(s)")
+        pre = layer_spec.prefix
+        self.scale = float(layer_spec.params.get("residual_scale", 1.0))
+        self.norms = [build_part("norm", s, pre + s.name) for s in layer_spec.norms]
+        if not all(hasattr(n, "join") for n in self.norms):
+            raise ValueError("the norms of a post_norm block must be able to join a branch and the stream")
+        self.mixer = build_part("mixer", layer_spec.mixer, pre + layer_spec.mixer.name)
+        self.feed_forward = None
+        if layer_spec.feed_forward is not None:
+            self.feed_forward = build_part("feed_forward", layer_spec.feed_forward,
+                                           pre + layer_spec.feed_forward.name)
+
+    parts, parameters, bind = SandwichBlock.parts, SandwichBlock.parameters, SandwichBlock.bind
+    supports_graph, cache_needs = SandwichBlock.supports_graph, SandwichBlock.cache_needs
+    streamed_weights = SandwichBlock.streamed_weights
+
+    def forward(self, ctx, stream: ResidualStream, cache) -> None:
+        if stream.pending is not None or stream.rows is None:
+            stream.rows = stream_rows(ctx, stream)
+        self.norms[0].join(ctx, stream, self.mixer.forward(ctx, stream.rows, cache), self.scale)
+        if self.feed_forward is not None:
+            self.norms[1].join(ctx, stream, self.feed_forward.forward(ctx, stream.rows), self.scale)
+
+
+register_part("arrangement", "post_norm", lambda layer_spec, name="": PostNormBlock(layer_spec))

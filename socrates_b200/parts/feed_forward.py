@@ -4,7 +4,8 @@ weights are bound their rows are interleaved (row 2f = gate_f, row 2f+1 = up_f),
 gate and its up value are neighbours in the product's output.  For many rows the
 tensor-core kernel then applies SiLU*mul in its epilogue and the [N, 2F] intermediate is
 never written; otherwise a SiLU*mul kernel reads the interleaved product.
-silu(z) = z * sigmoid(z) in float32."""
+silu(z) = z * sigmoid(z) in float32.  With `activation: "gelu_tanh"` the gate goes through the tanh form of gelu
+instead (GeGLU); everything else is the same."""
 
 from __future__ import annotations
 
@@ -24,6 +25,9 @@ class SwiGLU(Part):
         self.inter = int(spec.params["intermediate_size"])
         # tensor names after the part's prefix: gate, up, down (a plan may rename them)
         self.names = tuple(spec.params.get("names", ("gate_proj.weight", "up_proj.weight", "down_proj.weight")))
+        self.act = str(spec.params.get("activation", "silu"))
+        if self.act not in ops.GATE_ACTIVATIONS:
+            raise ValueError(f"unknown activation {self.act!r} of a gate; known: {sorted(ops.GATE_ACTIVATIONS)}")
         self.gate_up: Optional[Linear] = None
         self.down: Optional[Linear] = None
 
@@ -48,11 +52,11 @@ class SwiGLU(Part):
     def forward(self, ctx, x: torch.Tensor) -> Branch:
         N = x.shape[0]
         if ctx.can_fuse_silu_mul(N, self.gate_up.weight, x.dtype):
-            act = self.gate_up(ctx, x, "act", epilogue=1)
+            act = self.gate_up(ctx, x, "act", epilogue=1 + ops.GATE_ACTIVATIONS[self.act])
         else:
             gu = self.gate_up(ctx, x, "gate_up")
             act = ctx.buffers.take("act", N, (self.inter,), ctx.dtype)
-            ops.silu_mul(act, gu, interleaved=True)
+            ops.silu_mul(act, gu, interleaved=True, act=self.act)
         return Branch(self.down(ctx, act, "branch", out="partial"))
 
 

@@ -27,7 +27,7 @@ class Linear:
         product is cut along K (the weight-streaming regime), else the model dtype: for
         consumers that can add the parts themselves."""
         M = x.shape[0]
-        N = self.out_features // 2 if epilogue == 1 else self.out_features
+        N = self.out_features // 2 if epilogue else self.out_features
         if out == "model_or_partial":
             out = "partial" if ctx.gemm_splits(M, self.weight, x.dtype, shares=False) > 1 else "model"
         if out == "model":

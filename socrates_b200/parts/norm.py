@@ -50,6 +50,7 @@ def fold_and_norm(stream: ResidualStream, gain: Optional[torch.Tensor], out: Opt
     if row_index is None:
         stream.pending = None
         stream.add_rows = stream.add_vec = None
+        stream.rows = None
 
 
 class RMSNorm(Part):
@@ -80,6 +81,17 @@ class RMSNorm(Part):
         out = take(buffer, M, (self.dim,), out_dtype or ctx.dtype)
         fold_and_norm(stream, self.gain, out, self.eps, row_index)
         return out
+
+    def join(self, ctx, stream: ResidualStream, branch, scale: float) -> None:
+        """The stream becomes norm(scale * stream + branch): the float32 residual, and `stream.rows` in the model
+        dtype (the residual itself in the float32 engine)."""
+        if branch.post_gain is not None or branch.scale != 1.0 or branch.also is not None:
+            raise ValueError("a branch that joins before the norm is plain partial sums (and a bias)")
+        N, d = stream.residual.shape
+        out = None if ctx.dtype == torch.float32 else ctx.buffers.take("stream_rows", N, (d,), ctx.dtype)
+        ops.fold_rmsnorm(stream.residual, branch.partial, self.gain, out, self.eps, branch_bias=branch.bias,
+                         res_scale=scale, norm_residual=True)
+        stream.rows = stream.residual if out is None else out
 
 
 register_part("norm", "rmsnorm", RMSNorm)

@@ -6,6 +6,10 @@ context keeps its frequency, one that turns fewer than `slow` times gets frequen
 dims between are blended linearly by their index; every cosine and sine is then multiplied by
 `magnitude` = 0.1 ln(factor) + 1, which the rotation kernel takes as a constant.
 
+With `scaling: {"kind": "wavelength", ...}` (factor, low, high, original) each frequency f is judged by its
+wavelength l = 2 pi / f instead: l < original / high keeps f, l > original / low gets f / factor, and between the
+two f is (1 - s) f / factor + s f with s = (original / l - low) / (high - low); nothing else is scaled.
+
 A position encoding hands the mixer a float32 table `inv_freq[rotary_dim/2]` and the
 number of leading dims that rotate; the kernel computes angle = float32(position) *
 inv_freq[j] and pairs dim j with j + rotary_dim/2 (or, with `pairing: "neighbours"`, dim 2j
@@ -50,16 +54,25 @@ class Rotary(Part):
         self._low: Optional[torch.Tensor] = None
         self.scaling = spec.params.get("scaling")
         self.magnitude = 1.0                    # on every cosine and sine
+        self.by_wavelength = bool(self.scaling) and self.scaling.get("kind") == "wavelength"
         if self.scaling:
-            for key in ("factor", "original", "fast", "slow"):
+            for key in ("factor", "original", *(("low", "high") if self.by_wavelength else ("fast", "slow"))):
                 if key not in self.scaling:
                     raise ValueError(f"scaled rotation lacks {key!r}")
             if not float(self.scaling["factor"]) > 0:
                 raise ValueError("the scaling factor must be positive")
+            if self.by_wavelength and not float(self.scaling["high"]) > float(self.scaling["low"]) > 0:
+                raise ValueError("the scaling needs 0 < low < high")
+        if self.scaling and not self.by_wavelength:
             self.magnitude = 0.1 * math.log(float(self.scaling["factor"])) + 1.0
 
     def _scaled(self, f: torch.Tensor) -> torch.Tensor:
-        """Blend of f and f / factor by dim index (float64 in, float64 out)."""
+        """Blend of f and f / factor, by dim index or by wavelength (float64 in, float64 out)."""
+        if self.by_wavelength:
+            factor, low, high, original = (float(self.scaling[k]) for k in ("factor", "low", "high", "original"))
+            turns = original * f / (2.0 * math.pi)                       # original / wavelength
+            share = ((turns - low) / (high - low)).clamp(0.0, 1.0)       # of the unscaled frequency
+            return (1.0 - share) * f / factor + share * f
         sc, r = self.scaling, self.rotary_dim
         factor, original = float(sc["factor"]), float(sc["original"])
 

@@ -15,6 +15,11 @@ every token ID (no expert twice in a row), and each of them counts 1 / top.
 With `weighting: "chosen"` the experts are chosen by the logits themselves (plus `router.b` with `router_bias`)
 and weighed by the softmax over the chosen logits only.
 
+With `weighting: "sigmoid"` scores are s = sigmoid(z): a group counts with the sum of its two largest s, the `top`
+largest s of the open groups are chosen and weigh s / (their sum + 1e-20) * `scale`.
+
+With `unit: "relu_squared"` an expert has no gate: W_down relu(W_up x)^2.
+
 With `clamp` (`limit`, `alpha`, `offset`) an expert is the clamped gated unit instead:
     g = min(W_gate x, limit) ,  u = clamp(W_up x, -limit, limit) ,  W_down (g * sigmoid(alpha g) * (u + offset))
 and `shared` (`intermediate_size`, `limit`) names one more such expert that runs for every token with weight one:
@@ -30,7 +35,7 @@ recorded into graphs like any other; the price is that every expert is computed 
 costs nothing while a step streams the weights anyway (decoding) and E / top times the needed products
 for long prompt portions.
 For clamped experts gates and values are two halves of the first product and one kernel clamps, gates and
-scales all experts' units.
+scales all experts' units; experts without a gate have half the first product and one such kernel.
 Tensors: `<name>router`, `router.b`, `correction` (or `table`), `e<i>.gate`, `e<i>.up`, `e<i>.down`, `shared.gate`,
 `shared.up`, `shared.down`.
 """
@@ -78,9 +83,19 @@ class RoutedFeedForward(Part):
             raise ValueError(f"{self.E} router outputs in {self.groups} groups of which {self.keep} stay")
         if not 1 <= self.top <= self.keep * (self.E // self.groups):
             raise ValueError(f"{self.top} choices among {self.keep * (self.E // self.groups)} open experts")
-        self.weighting = str(p.get("weighting", "all"))       # softmax over "all" outputs or the "chosen" ones
-        if self.weighting not in ("all", "chosen"):
-            raise ValueError(f"weighting {self.weighting!r} is neither 'all' nor 'chosen'")
+        self.weighting = str(p.get("weighting", "all"))       # softmax over "all" outputs or the "chosen" ones, or "sigmoid"
+        if self.weighting not in ("all", "chosen", "sigmoid"):
+            raise ValueError(f"weighting {self.weighting!r} is none of 'all', 'chosen' and 'sigmoid'")
+        if self.weighting == "sigmoid" and (self.routing == "table" or self.correction_tensor):
+            raise ValueError("weights from sigmoid scores take no table and no correction")
+        self.scale = float(p.get("scale", 1.0))
+        if self.scale != 1.0 and self.weighting != "sigmoid":
+            raise ValueError("a scale on the weights is served with sigmoid scores only")
+        self.unit = str(p.get("unit", "gated"))
+        if self.unit not in ("gated", "relu_squared"):
+            raise ValueError(f"an expert's unit {self.unit!r} is neither 'gated' nor 'relu_squared'")
+        if self.unit != "gated" and (p.get("clamp") is not None or p.get("shared")):
+            raise ValueError("experts without a gate take no clamp and no shared expert")
         if self.weighting == "chosen" and (self.routing == "table" or self.groups > 1 or self.correction_tensor):
             raise ValueError("weights from the chosen logits take no table, groups or correction")
         self.router_bias = bool(p.get("router_bias", False))
@@ -114,7 +129,8 @@ class RoutedFeedForward(Part):
             out[n + "shared.up"] = ParamSpec((self.shared_inter, self.hidden))
             out[n + "shared.down"] = ParamSpec((self.hidden, self.shared_inter))
         for e in range(self.experts):
-            out[f"{n}e{e}.gate"] = ParamSpec((self.inter, self.hidden))
+            if self.unit == "gated":
+                out[f"{n}e{e}.gate"] = ParamSpec((self.inter, self.hidden))
             out[f"{n}e{e}.up"] = ParamSpec((self.inter, self.hidden))
             out[f"{n}e{e}.down"] = ParamSpec((self.hidden, self.inter))
         return out
@@ -134,6 +150,10 @@ class RoutedFeedForward(Part):
             names = [f"{n}e{e}." for e in range(self.experts)] + ([n + "shared."] if self.shared_inter else [])
             self.gate_up = Linear(torch.cat([tensors[x + "gate"] for x in names] + [tensors[x + "up"] for x in names], dim=0))
             self.down = Linear(torch.cat([tensors[x + "down"] for x in names], dim=1))
+            return
+        if self.unit != "gated":
+            self.gate_up = Linear(torch.cat([tensors[f"{n}e{e}.up"] for e in range(self.experts)], dim=0))
+            self.down = Linear(torch.cat([tensors[f"{n}e{e}.down"] for e in range(self.experts)], dim=1))
             return
         rows = [torch.stack([tensors[f"{n}e{e}.gate"], tensors[f"{n}e{e}.up"]], dim=1).reshape(2 * F, d)
                 for e in range(self.experts)]
@@ -157,6 +177,10 @@ class RoutedFeedForward(Part):
         if self.weighting == "chosen":
             ops.moe_router(x, self.router, self.bias, weights, ids, picked, self.top)
             return weights, ids, picked
+        if self.weighting == "sigmoid":
+            ops.moe_router(x, self.router, None, weights, ids, picked, self.top, sigmoid=True, groups=self.groups,
+                           keep=self.keep, scale=self.scale)
+            return weights, ids, picked
         logits = take("moe_logits", N, (self.E,), torch.float32)
         ops.moe_logits(logits, x, self.router)
         ops.moe_route(logits, self.correction, weights, ids, picked, self.groups, self.keep, self.top)
@@ -172,13 +196,17 @@ class RoutedFeedForward(Part):
             ops.moe_glu_clamp(act, gu, weights, self.experts, self.inter, limit,
                               float(self.shared["limit"]) if self.shared else limit, float(self.clamp["alpha"]),
                               float(self.clamp["offset"]))
+        elif self.unit != "gated":
+            up = self.gate_up(ctx, x, "moe_gate_up", out="model_or_partial")
+            act = ctx.buffers.take("moe_act", N, (width,), ctx.dtype)
+            ops.moe_act(act, up, weights, self.experts, self.inter)
         elif ctx.can_fuse_silu_mul(N, self.gate_up.weight, x.dtype):
             act = self.gate_up(ctx, x, "moe_act", epilogue=1)
         else:
             gu = self.gate_up(ctx, x, "moe_gate_up")
             act = ctx.buffers.take("moe_act", N, (width,), ctx.dtype)
             ops.silu_mul(act, gu, interleaved=True)
-        if self.clamp is None:
+        if self.clamp is None and self.unit == "gated":
             ops.moe_scale(act, weights, self.experts)
         S = ctx.gemm_splits(N, self.down.weight, act.dtype)
         slabs = S + (1 if self.identity else 0)
