@@ -493,6 +493,26 @@ def _samovik(width, heads):
             "token_side": {"dim": width // 8}, "layers": [lat, lin, lin, wkv] * 2}
 
 
+def _kusirax(width, heads):
+    """A Kusirax configuration at real layer widths, eight layers: token-shift mixing with heads of 64, attention with
+    heads of 128 (half of the dims rotate), twice attention in chunks of 1,024 with capped scores and slopes, all twice;
+    heads / 4 key/value heads as in the Qwen3 shape, values blended in every attention layer.  Dense gelu-gated
+    feed-forwards of four times the width and sixteen experts of one width, four of them a token, take turns."""
+    dense = {"kind": "dense", "ff": 4 * width}
+    moe = {"kind": "moe", "expert": {"ff": width},
+           "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}, "scale": 2.0}}
+    kv = max(1, heads // 4)
+    wkv = {"type": "wkv", "mlp": dense, "mixer": {"heads": 2 * heads, "dim": 64}}
+    att = {"type": "attention", "mlp": moe, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+        "rot": {"base": 5e5, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    cut = {"type": "attention_2", "mlp": dense, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True, "softcap": 30.0,
+        "mask": {"size": 1024}}}
+    return {"architecture": "Kusirax", "vocab": 32000, "width": width, "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
+            "layers": [wkv, att, cut, dict(cut, mlp=moe)] * 2}
+
+
 def _qwen3_like(width, runs, heads):
     """The Qwen3 decoder at the same width, number of layer runs, head size and feed-forward width."""
     return {"architectures": ["Qwen3ForCausalLM"], "vocab_size": 32000, "hidden_size": width,
@@ -502,9 +522,10 @@ def _qwen3_like(width, runs, heads):
 
 
 def run_compare(args):
-    """`--compare bofusun|loletar|samerax|magedra|samovik`: prefill and decode throughput of another design at real layer
-    widths (random weights) beside the Qwen3 decoder at equal width, layer runs and head size (Samovik: and beside
-    Loletar, whose layers carry routed experts and a matrix recurrence as well).  One JSON line."""
+    """`--compare bofusun|loletar|samerax|magedra|samovik|kusirax`: prefill and decode throughput of another design at
+    real layer widths (random weights) beside the Qwen3 decoder at equal width, layer runs and head size (Samovik: and
+    beside Loletar, whose layers carry routed experts and a matrix recurrence as well; Kusirax: and beside Samovik,
+    which has the same recurrence and routed experts).  One JSON line."""
     import torch
 
     from socrates_b200 import Engine
@@ -527,13 +548,14 @@ def run_compare(args):
         design = args.compare
         bof = {"bofusun": lambda: _bofusun(width, 5, heads, 1024), "loletar": lambda: _loletar(width, heads),
                "samerax": lambda: _samerax(width, heads), "magedra": lambda: _magedra(width, heads),
-               "samovik": lambda: _samovik(width, heads)}[design]()
+               "samovik": lambda: _samovik(width, heads), "kusirax": lambda: _kusirax(width, heads)}[design]()
         runs = len(config_from_dict(bof).plan().order)
         only = [x for x in (args.only.split(",") if args.only else [design, "qwen3"])]
         beside = [(design, bof), ("qwen3", _qwen3_like(width, runs, heads))]
-        if design == "samovik":
-            beside.insert(1, ("loletar", _loletar(width, heads)))
-            only = only if args.only else [design, "loletar", "qwen3"]
+        third = {"samovik": ("loletar", _loletar), "kusirax": ("samovik", _samovik)}.get(design)
+        if third is not None:
+            beside.insert(1, (third[0], third[1](width, heads)))
+            only = only if args.only else [design, third[0], "qwen3"]
         for label, cfg_dict in beside:
             if label not in only:
                 continue
@@ -603,7 +625,7 @@ def run_compare(args):
             "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak",
             "vs_baseline": None, "dtype": "bf16",
             "data": "synthetic: random weights, token ids uniform over the vocabulary",
-            "config": {"model": f"{args.compare.capitalize()} and {'Loletar and ' if args.compare == 'samovik' else ''}Qwen3 decoders "
+            "config": {"model": f"{args.compare.capitalize()} and {(third[0].capitalize() + ' and ') if third else ''}Qwen3 decoders "
                                 f"at equal width and layer runs", "global_batch": B,
                        "seq_len": ctx, "prefill_tokens": T, "parallelism": "single GPU", "cuda_graph": True,
                        "l2": "inputs larger than L2 at widths 2k and 4k; a step's weights at 1k are not"},
@@ -658,8 +680,8 @@ def main():
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-prefill", action="store_true")
-    ap.add_argument("--compare", default=None, choices=("bofusun", "loletar", "samerax", "magedra", "samovik"),
-                    help="the Bofusun, the Loletar, the Samerax, the Magedra or the Samovik design at real layer widths beside Qwen3 at "
+    ap.add_argument("--compare", default=None, choices=("bofusun", "loletar", "samerax", "magedra", "samovik", "kusirax"),
+                    help="the Bofusun, the Loletar, the Samerax, the Magedra, the Samovik or the Kusirax design at real layer widths beside Qwen3 at "
                          "equal size "
                          "(prefill and decode); the default workload is not run")
     ap.add_argument("--only", default=None, help="with --compare: run only these of the pair, e.g. 'loletar' or 'qwen3'")

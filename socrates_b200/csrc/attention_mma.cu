@@ -157,7 +157,7 @@ template <int NBQ> struct ColumnMap {
     sb::RowScores row[2 * NBQ];
     int pos;
     __device__ __forceinline__ float operator()(float s, int key, int nb, int e) const {
-        return row[2 * nb + e](s, (float)(key - pos));
+        return row[2 * nb + e](s, (float)(key - pos));     // an exact distance
     }
 };
 
@@ -203,8 +203,10 @@ attn_decode_kernel(bf16* __restrict__ out, float* __restrict__ part_o, float* __
     if constexpr (MAPPED) {                                 // the thread's columns are query heads 2 (lane % 4), + 1
         col_map.pos = pos;
 #pragma unroll
-        for (int c = 0; c < 2 * NBQ; ++c)
+        for (int c = 0; c < 2 * NBQ; ++c) {
             col_map.row[c].set(score_map, scale_log2, h0 + min(G - 1, 8 * (c >> 1) + 2 * (lane & 3) + (c & 1)));
+            col_map.row[c].from(0.f);
+        }
     }
 
     const bool empty = k_begin >= k_end;                    // an empty partition (only when NP > 1)

@@ -188,7 +188,7 @@ constexpr int THREADS = ROWS + 96;
 // MAPPED: scores are capped and / or lose a slope times the distance (see score_map.cuh); `scale_log2` is the
 // plain scale then, and a row's scores are turned into units of log2 as they are read.
 template <int D, bool MAPPED>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
                             bf16* __restrict__ out, const bf16* __restrict__ q,
                             const int* __restrict__ block_table, int table_width,
@@ -431,9 +431,14 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
                 for (int j = 0; j < 32; ++j) s[32 + j] = __uint_as_float(raw[j]);
             }
             if constexpr (MAPPED) {
-                const float ahead = (float)(tile_start - qpos);
+                row_scores.from((float)(tile_start - qpos));
+                if (row_scores.capped) {
 #pragma unroll
-                for (int j = 0; j < 64; ++j) s[j] = row_scores(s[j], ahead + (float)j);
+                    for (int j = 0; j < 64; ++j) s[j] = row_scores.with_cap(s[j], (float)j);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 64; ++j) s[j] = row_scores.plain(s[j], (float)j);
+                }
             }
             // position masks only where some row of the block cannot see some key of the tile;
             // rows past the tile (qpos = -1) are masked by the same test

@@ -24,12 +24,12 @@ __host__ __device__ __forceinline__ int first_visible(int pos, int window, int c
 }
 
 // One query row's constants of the map, for scores in units of log2 (softmax weights are 2^s then):
-//   capped:   cap * tanh(z) = cap - 2 cap / (1 + e^{2z}), z = raw * scale / cap, in hardware ex2 and division.
+//   capped:   cap * tanh(z) = cap - 2 cap / (1 + e^{2z}), z = raw * scale / cap, in hardware ex2 and reciprocal.
 //             Its absolute error is a few 1e-7 of the cap, whatever the score's size.
 //   otherwise raw * scale.
 // and then + slope * (j - i).
 struct RowScores {
-    float in, cap, slope;
+    float in, cap, slope, base;
     bool capped;
 
     __device__ __forceinline__ void set(const ScoreMap& m, float scale, int h) {
@@ -38,14 +38,20 @@ struct RowScores {
         cap = m.cap * LOG2;
         in = capped ? scale / m.cap * (2.0f * LOG2) : scale * LOG2;
         slope = m.slopes != nullptr ? m.slopes[h] * LOG2 : 0.f;
+        base = 0.f;
     }
-    // `ahead` = key position - query position
-    __device__ __forceinline__ float operator()(float raw, float ahead) const {
-        const float base = slope * ahead;
-        if (!capped) return fmaf(raw, in, base);
-        float e;
+    // the keys that follow are counted from one that is `ahead` = key position - query position away
+    __device__ __forceinline__ void from(float ahead) { base = fmaf(slope, ahead, capped ? cap : 0.f); }
+
+    __device__ __forceinline__ float plain(float raw, float offset) const { return fmaf(raw, in, fmaf(slope, offset, base)); }
+    __device__ __forceinline__ float with_cap(float raw, float offset) const {
+        float e, r;
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * in));
-        return fmaf(-2.0f * cap, __fdividef(1.0f, 1.0f + e), cap + base);
+        asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+        return fmaf(-2.0f * cap, r, fmaf(slope, offset, base));
+    }
+    __device__ __forceinline__ float operator()(float raw, float offset) const {
+        return capped ? with_cap(raw, offset) : plain(raw, offset);
     }
 };
 
