@@ -704,7 +704,7 @@ static void qk_launch(const void* qkv, const float* parts, int S, size_t part_st
                       int spread, cudaStream_t stream) {
     const int n_heads = Hq + 2 * Hkv;
     const bool plain = (rotary_dim == D || rotary_dim == 0) && !extra.any();
-    const bool fast = (plain || rotary_dim % (D / 8) == 0) && (D == 64 || D == 128 || D == 256) && Dv == D &&
+    const bool fast = (D == 64 || D == 128 || D == 256) && (plain || rotary_dim % (D / 8) == 0) && Dv == D &&
                       row_width == n_heads * D && !(neighbours && rotary_dim > 0) && sub == D && magnitude == 1.0f &&
                       !spread && (reinterpret_cast<uintptr_t>(extra.bias) & 15) == 0;
     // Heads per block: 4 (a head per warp) while that still fills the GPU, more for long batches.
