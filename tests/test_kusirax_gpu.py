@@ -128,7 +128,7 @@ def test_stream_after_every_layer(tmp_path, dtype, name):
         C.StepContext.__init__ = original
     assert len(got) == len(want) == len(cfg["layers"])
     for i, (a, b) in enumerate(zip(got, want)):
-        assert part_err(a, b) < (1e-4 if dtype == torch.float32 else 4e-2), i
+        assert part_err(a, b) < (1e-4 if dtype == torch.float32 else 6e-2), i
 
 
 # ------------------------------------------------------------------------------------------
@@ -406,7 +406,7 @@ def test_a_prompt_of_many_segments(models, dtype):
 # the entry point, the scheduler, the command line, the replay
 
 @pytest.mark.parametrize("dtype,graphs", [("float32", False), ("bfloat16", True)])
-@pytest.mark.parametrize("name", ["A", "B", "C", "E", "F"])
+@pytest.mark.parametrize("name", ["A", "B", "C", "E", "F", "G"])
 def test_greedy_generation_through_the_entry_point(models, name, dtype, graphs):
     """Five requests through Engine: queued, admitted as rows come free, prompts cut by the token budget, decoded side
     by side (bfloat16: through recorded graphs), 60 new tokens each.  Every produced token is the plain statement's
