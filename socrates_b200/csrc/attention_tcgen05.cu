@@ -185,9 +185,14 @@ __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
 // that issues the P.V products
 constexpr int THREADS = ROWS + 96;
 
-// MAPPED: scores are capped and / or lose a slope times the distance (see score_map.cuh); `scale_log2` is the
+// MAPPED 1: scores are capped and / or lose a slope times the distance (see score_map.cuh); `scale_log2` is the
 // plain scale then, and a row's scores are turned into units of log2 as they are read.
-template <int D, bool MAPPED>
+// MAPPED 2: the same with a cap of at most BOUND_LOG2 in units of log2.  A row's largest score then lies between minus and
+// plus the cap (the query's own position costs no slope), so 2^score itself is a weight that float32 holds with its sums:
+// no running maximum, no rescaling, and every score becomes its weight on its own.
+constexpr float BOUND_LOG2 = 80.0f;
+
+template <int D, int MAPPED>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
                             bf16* __restrict__ out, const bf16* __restrict__ q,
@@ -405,8 +410,8 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
         const int qpos = tok < n_tok ? first_pos + tok : -1;   // rows past the tile see no key
         const int qlo = qpos >= 0 ? first_visible(qpos, window, map.chunk) : 0;
         RowScores row_scores;
-        if constexpr (MAPPED) row_scores.set(map, scale_log2, kh * G + g);
-        const float per_unit = MAPPED ? 1.0f : scale_log2;     // from the scores below to exponents of 2
+        if constexpr (MAPPED != 0) row_scores.set(map, scale_log2, kh * G + g);
+        const float per_unit = MAPPED != 0 ? 1.0f : scale_log2;     // from the scores below to exponents of 2
         const uint32_t lane_base = tmem + (static_cast<uint32_t>(warp * 32) << 16);
         bool ok = true;
         for (int i = 0; i < n_tiles; ++i) {
@@ -430,12 +435,12 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
 #pragma unroll
                 for (int j = 0; j < 32; ++j) s[32 + j] = __uint_as_float(raw[j]);
             }
-            if constexpr (MAPPED) {
+            if constexpr (MAPPED != 0) {
                 row_scores.from((float)(tile_start - qpos));
-                if (row_scores.capped) {
+                if (MAPPED == 1 && row_scores.capped) {
 #pragma unroll
                     for (int j = 0; j < 64; ++j) s[j] = row_scores.with_cap(s[j], (float)j);
-                } else {
+                } else if (MAPPED == 1) {
 #pragma unroll
                     for (int j = 0; j < 64; ++j) s[j] = row_scores.plain(s[j], (float)j);
                 }
@@ -444,6 +449,37 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
             // rows past the tile (qpos = -1) are masked by the same test
             const bool masked = i < keep_tiles ? (tile_start + KTILE > kf || n_tok < TQ)
                                                : (tile_start + KTILE - 1 > first_pos || tile_start < last_qlo || n_tok < TQ);
+            // weights (of key j of the tile: weight(j)), their sum, and their two terms over the scores of this very row,
+            // all 64 of which were read into registers above
+            auto write_weights = [&](auto weight) {
+                float l4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int c = 0; c < KTILE; c += 32) {
+                    uint32_t ph[16], pl[16];
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        const float p0 = weight(c + 2 * j);
+                        const float p1 = weight(c + 2 * j + 1);
+                        l4[j & 3] += p0 + p1;
+                        const uint32_t h = pack_bf16(p0, p1);
+                        ph[j] = h;
+                        pl[j] = pack_bf16(p0 - __uint_as_float(h << 16), p1 - __uint_as_float(h & 0xffff0000u));
+                    }
+                    tmem_st16(lane_base + COL_SP + 64 * b + (c >> 1), ph);
+                    tmem_st16(lane_base + COL_SP + 64 * b + 32 + (c >> 1), pl);
+                }
+                l_run += (l4[0] + l4[1]) + (l4[2] + l4[3]);
+            };
+            if constexpr (MAPPED == 2) {
+                if (masked)
+                    write_weights([&](int j) {
+                        const int kpos = tile_start + j;
+                        const float p = ex2_approx(row_scores.with_cap(s[j], (float)j));
+                        return (kpos <= qpos && (kpos >= qlo || kpos < kf)) ? p : 0.f;
+                    });
+                else
+                    write_weights([&](int j) { return ex2_approx(row_scores.with_cap(s[j], (float)j)); });
+            } else {
             if (masked) {
 #pragma unroll
                 for (int j = 0; j < 64; ++j) {
@@ -493,24 +529,8 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
             }
             // p = 2^((s - m) * scale) as one multiply-add and one ex2; masked scores are -inf -> 0
             const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref * per_unit;
-            float l4[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int c = 0; c < KTILE; c += 32) {
-                uint32_t ph[16], pl[16];
-#pragma unroll
-                for (int j = 0; j < 16; ++j) {
-                    const float p0 = ex2_approx(fmaf(s[c + 2 * j], per_unit, neg_m));
-                    const float p1 = ex2_approx(fmaf(s[c + 2 * j + 1], per_unit, neg_m));
-                    l4[j & 3] += p0 + p1;
-                    const uint32_t h = pack_bf16(p0, p1);
-                    ph[j] = h;
-                    pl[j] = pack_bf16(p0 - __uint_as_float(h << 16), p1 - __uint_as_float(h & 0xffff0000u));
-                }
-                // over the scores of this very row: all 64 were read into registers above
-                tmem_st16(lane_base + COL_SP + 64 * b + (c >> 1), ph);
-                tmem_st16(lane_base + COL_SP + 64 * b + 32 + (c >> 1), pl);
+            write_weights([&](int j) { return ex2_approx(fmaf(s[j], per_unit, neg_m)); });
             }
-            l_run += (l4[0] + l4[1]) + (l4[2] + l4[3]);
             tmem_st_wait();
             // slots of this tile outside [lo, hi): zero their V rows (thread j < 64 owns key j)
             if (tile_start < lo || tile_start + KTILE > hi) {
@@ -626,7 +646,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_k, const __g
     }
 }
 
-template <int D, bool MAPPED>
+template <int D, int MAPPED>
 int launch(const CUtensorMap& mk, const CUtensorMap& mv, void* out, const void* q, const int* block_table,
            int table_width, const int* seq_starts, const int* seq_rows, const int* seq_first_pos, int R, int N,
            int Hq, int Hkv, int BS, int window, float scale, int* status, const void* gate, long long gate_stride,
@@ -645,8 +665,8 @@ int launch(const CUtensorMap& mk, const CUtensorMap& mv, void* out, const void* 
     dim3 grid((N / TQ + R) * Hkv);                           // an upper bound of the number of tiles, times heads
     sb::launch(kernel, grid, dim3(THREADS), smem_bytes<D>() + table_width * 4, stream, mk, mv, (bf16*)out,
                (const bf16*)q, block_table, table_width, seq_starts, seq_rows, seq_first_pos, R, Hq, Hkv, BS, window,
-               MAPPED ? scale : scale * LOG2E, status, (const bf16*)gate, gate_stride, gate_per_dim, has_sink,
-               has_sink ? (MAPPED ? sink * LOG2E : sink / scale) : 0.f, keep_first, out_f32, map);
+               MAPPED != 0 ? scale : scale * LOG2E, status, (const bf16*)gate, gate_stride, gate_per_dim, has_sink,
+               has_sink ? (MAPPED != 0 ? sink * LOG2E : sink / scale) : 0.f, keep_first, out_f32, map);
     return 0;
 }
 
@@ -698,8 +718,9 @@ extern "C" int sb_attention_prefill_tcgen05(void* out, const void* q, const void
                         page_size, window, scale, status, gate, gate_stride, gate_per_dim, has_sink, sink, keep_first, \
                         out_f32, map, stream)
     int rc;
-    if (map.maps_scores()) rc = D == 64 ? SB_TILE(64, true) : SB_TILE(128, true);
-    else rc = D == 64 ? SB_TILE(64, false) : SB_TILE(128, false);
+    if (cap > 0.f && cap * LOG2E <= BOUND_LOG2 && !has_sink) rc = D == 64 ? SB_TILE(64, 2) : SB_TILE(128, 2);
+    else if (map.maps_scores()) rc = D == 64 ? SB_TILE(64, 1) : SB_TILE(128, 1);
+    else rc = D == 64 ? SB_TILE(64, 0) : SB_TILE(128, 0);
 #undef SB_TILE
     if (rc != 0) return rc;
     SB_LAUNCH_CHECK();

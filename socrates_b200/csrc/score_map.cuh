@@ -11,7 +11,7 @@ namespace sb {
 
 struct ScoreMap {
     float cap;              // 0: not capped
-    const float* slopes;    // [Hq] or null
+    const float* slopes;    // [Hq], not negative, or null
     int chunk;              // 0: no chunks
 
     __host__ __device__ bool maps_scores() const { return cap > 0.f || slopes != nullptr; }

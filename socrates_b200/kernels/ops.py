@@ -392,7 +392,7 @@ def attention_decode_mma(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tenso
     `variant` picks the kernel's (warps, stages); 0 is the default.  2 to 4 partitions are
     merged inside the kernel (a thread-block cluster per token and KV head), more by a
     reduce kernel through the scratch buffers.  `softcap` (0: none): s = c * tanh(s / c); `slopes` float32
-    [Hq]: a key loses slope * distance; `chunk` > 0: only keys of the query's own chunk of so many positions.
+    [Hq], not negative: a key loses slope * distance; `chunk` > 0: only keys of the query's own chunk of so many positions.
 
     The kernel reads the block table, rows, positions and the keys and values below each
     position before it waits for the kernel that precedes it on the stream: those must be

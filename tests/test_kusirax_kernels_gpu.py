@@ -56,7 +56,7 @@ class Paged:
 
 MAPS = [dict(cap=0.0, slopes=False, chunk=0), dict(cap=2.5, slopes=False, chunk=0), dict(cap=0.0, slopes=True, chunk=0),
         dict(cap=0.0, slopes=False, chunk=20), dict(cap=4.0, slopes=True, chunk=48), dict(cap=1.5, slopes=True, chunk=7),
-        dict(cap=30.0, slopes=True, chunk=100)]
+        dict(cap=30.0, slopes=True, chunk=100), dict(cap=60.0, slopes=True, chunk=48)]
 
 
 def case(H, G, dk, dv, dtype, m, seed):
@@ -137,6 +137,30 @@ def test_cuda_core_attention_with_mapped_scores(shape, m, dtype):
         ops.attention_bias_tile(out, qd, pages.k_pool, pages.v_pool, pages.table, i32(starts), i32([0, 1, 2]), i32(firsts), H,
                                 scale, **kw)
         assert err(out.double().cpu(), want) < tol
+
+
+@pytest.mark.parametrize("cap", [50.0, 55.0, 70.0])
+@pytest.mark.parametrize("sign", [-1.0, 1.0])
+def test_scores_at_the_cap(cap, sign):
+    """Every key of a row at minus the cap, or at plus the cap, but for one key a little off it: weights that take the
+    running maximum's place must neither vanish nor overflow."""
+    from socrates_b200.kernels import ops
+    g = torch.Generator().manual_seed(1)
+    n, H, D = 150, 2, 64
+    pages = Paged([n], 1, D, D, torch.bfloat16, g)
+    u = torch.ones(D)
+    k = (u[None] * 4.0 * (1 + 0.2 * torch.rand(n, 1, generator=g))).bfloat16()
+    k[20] = (u * sign * -1.0).bfloat16()                # this one alone is far from the rest for its queries
+    pages.k[0] = k[:, None]
+    for p in range(n):
+        pages.k_pool[int(pages.table[0, p // 16]), 0, p % 16] = k[p].to(DEV)
+    q = (sign * u[None, None] * torch.linspace(2.0, 4.0, n)[:, None, None]).repeat(1, H, 1).bfloat16()
+    slopes = torch.tensor([0.0, 0.3], dtype=F64)
+    want = attend(q.double(), pages.k[0].double(), pages.v[0].double(), range(n), 0.4, cap, slopes, 0)
+    out, status = torch.empty(n, H * D, dtype=torch.bfloat16, device=DEV), i32([0])
+    ops.attention_prefill_tcgen05(out, q.reshape(n, -1).to(DEV), pages.k_pool, pages.v_pool, pages.table, i32([0, n]), i32([0]),
+                                  i32([0]), H, 0.4, status, softcap=cap, slopes=slopes.float().to(DEV))
+    assert int(status.item()) == 0 and err(out.double().cpu(), want) < 8e-3
 
 
 def test_far_keys_keep_an_exact_slope():
