@@ -6,6 +6,8 @@
     python bench.py --compare loletar [--sizes 1k,2k,4k]
     python bench.py --compare samerax [--sizes 1k,2k,4k]
     python bench.py --compare magedra [--sizes 1k,2k,4k]
+    python bench.py --compare samovik [--sizes 1k,2k,4k]
+    python bench.py --compare kusirax [--sizes 1k,2k,4k]
 
 Default run: the layer sizes of the Qwen3-4B shape (36 layers, hidden 2560, 32 query
 heads over 8 KV heads, head_dim 128, intermediate 9728, vocabulary 151936, tied head),
